@@ -54,11 +54,16 @@ int llark_gemm(const void* A, int a_mn_major, long long lda, const void* B, int 
  *                         apply_rotary_pos_emb reached from m2t/models/llamav2.py:224; replaces llark_rope(inverse=0)
  *   LLARK_EPI_SWIGLU_BWD  acc = d(act) of the down projection's dgrad; a = gu bf16 [M, ld] (gate | up, N apart);
  *                         C[:, c] = dgate, C[:, N + c] = dup (C is dgu [M, ldc >= 2N]); replaces llark_swiglu_bwd
- * Results are bit-identical to the unfused sequences (same bf16 rounding points). */
+ * Results are bit-identical to the unfused sequences (same bf16 rounding points).
+ *   LLARK_EPI_RELU2       C = relu(acc + bias)^2, rounded once
+ *   LLARK_EPI_RELU_GLU    the rows of B alternate gate, up: C bf16 [M, N / 2], C[:, c] = relu(z[:, 2c]) * z[:, 2c + 1] with
+ *                         z = acc + bias, rounded once */
 /*   LLARK_EPI_SEGMENTS    not an epilogue: the rows of A / C come in runs that each multiply their own block of B (stacked
  *                         [i1, N, K]); a = device int triples (block, first row, rows <= 256), i0 = their number (an upper
- *                         bound when b points at a device word with the real number). Used by llark_gemm_segments. */
-enum { LLARK_EPI_NONE = 0, LLARK_EPI_QUICK_GELU = 1, LLARK_EPI_ROPE = 2, LLARK_EPI_SWIGLU_BWD = 3, LLARK_EPI_SEGMENTS = 4 };
+ *                         bound when b points at a device word with the real number), ld = LLARK_EPI_NONE or
+ *                         LLARK_EPI_RELU2. Used by llark_gemm_segments. */
+enum { LLARK_EPI_NONE = 0, LLARK_EPI_QUICK_GELU = 1, LLARK_EPI_ROPE = 2, LLARK_EPI_SWIGLU_BWD = 3, LLARK_EPI_SEGMENTS = 4,
+       LLARK_EPI_RELU2 = 5, LLARK_EPI_RELU_GLU = 6 };
 typedef struct LlarkGemmEpilogue {
     int kind;
     const void* a;
@@ -298,12 +303,24 @@ int llark_seq_gated_norm_add(const float* x, const float* y, const float* gate, 
 int llark_seq_rmsnorm_rows(const float* x, const int* rows, const float* w, void* out, int n_rows, int C, float eps,
                            int act_fp32, cudaStream_t stream);
 int llark_seq_relu2(const void* u, void* y, long long n, int act_fp32, cudaStream_t stream);
-/* C[M,N] = A[M,K] W[N,K]^T (+ bias fp32[N]), fp32 accumulation, A / W bf16 or (in_fp32) float, C float if c_fp32.
- * _rows: weight-streaming, for a handful of rows (decode). _simt: tiled, any shape, true fp32 when in_fp32. */
+/* out[i] = tanh(alpha * x[rows[i]]) * w + b in the activation dtype (rows == NULL: row i). */
+int llark_seq_tanh_norm(const float* x, const int* rows, float alpha, const float* w, const float* b, void* out, int n_rows,
+                        int C, int out_fp32, cudaStream_t stream);
+/* x_out = x + tanh(alpha * f) * w + b with f = y (optional) + sum_{k < top} wts[t, k] * z[pos_of[t * top + k]]; when x_act
+ * != NULL it also receives tanh(next_alpha * x_out) * next_w + next_b in the activation dtype. */
+int llark_seq_tanh_norm_add(const float* x, const float* y, const float* z, const int* pos_of, const float* wts, int top,
+                            float alpha, const float* w, const float* b, float next_alpha, const float* next_w,
+                            const float* next_b, float* x_out, void* x_act, long long rows, int C, int act_fp32,
+                            cudaStream_t stream);
+/* C[M,N] = act(A[M,K] W[N,K]^T (+ bias fp32[N])), fp32 accumulation, A / W bf16 or (in_fp32) float, C float if c_fp32.
+ * _rows: weight-streaming, for a handful of rows (decode). _simt: tiled, any shape, true fp32 when in_fp32.
+ * act: LLARK_ACT_RELU2 = relu(z)^2; LLARK_ACT_RELU_GLU = the rows of W alternate gate, up and C [M, N / 2] gets
+ * relu(z[:, 2c]) * z[:, 2c + 1]. */
+enum { LLARK_ACT_NONE = 0, LLARK_ACT_RELU2 = 1, LLARK_ACT_RELU_GLU = 2 };
 int llark_linear_rows(const void* A, long long lda, const void* W, long long ldw, void* C, long long ldc, int c_fp32,
-                      const float* bias, int M, int N, int K, int in_fp32, cudaStream_t stream);
+                      const float* bias, int M, int N, int K, int in_fp32, int act, cudaStream_t stream);
 int llark_linear_simt(const void* A, long long lda, const void* W, long long ldw, void* C, long long ldc, int c_fp32,
-                      const float* bias, int M, int N, int K, int in_fp32, cudaStream_t stream);
+                      const float* bias, int M, int N, int K, int in_fp32, int act, cudaStream_t stream);
 /* Per-head RMS norm of the q (H heads at column q_off) and k (G heads at k_off) parts of src fp32 [n_tok, ld] with
  * weights wq, wk fp32 [D]: qn [n_tok, H, D], kn [n_tok, G, D], vraw = the un-normed k. kring / vring non-NULL: also
  * written to ring entry position % cap of the request's slot (only when every request brings one token). */
@@ -322,12 +339,13 @@ int llark_seq_qkv_headnorm(const float* src, long long ld, int q_off, int k_off,
  * (G*D) projection with weights of that size. qk_freq fp32 [n_rot / 2]: the first n_rot entries of every q / k head are
  * rotated by position * qk_freq[i], pairs (i, i + n_rot/2) or, qk_interleaved, (2i, 2i + 1). v_freq fp32 [E / 2] (optional):
  * every value head is rotated the same way over all of E. Results in the activation dtype; with kring / vring the k / v rows
- * also go to ring entry position % cap of the slot. */
+ * also go to ring entry position % cap of the slot. unit (without wq): every rotated q / k head is divided by
+ * sqrt(mean(head^2) + eps). G = 0: queries only. */
 int llark_seq_qkv_rotary(const float* src, long long ld, int q_off, int k_off, int v_off, const float* wq, const float* wk,
                          const float* qk_freq, int n_rot, int qk_interleaved, const float* v_freq, int v_interleaved,
                          void* qn, void* kn, void* vv, void* kring, void* vring, const int* tok_seq, const int* cu,
                          const int* pos0, const int* slot, int n_tok, int H, int G, int D, int E, int cap, float eps,
-                         int act_fp32, cudaStream_t stream);
+                         int unit, int act_fp32, cudaStream_t stream);
 /* Sliding-window softmax attention: query at position i sees keys j with 0 <= i - j < window. Keys / values of this
  * step come from kn / vv ([n_tok, G, D] / [n_tok, G, E]), earlier ones from the rings [slots, cap, G, D|E] (entry
  * j % cap); from_ring_only = 1: the step's own token is already in the ring. score = q.k * scale_h[h]; the output is
@@ -435,10 +453,11 @@ int llark_seq_head_linear(const void* x, int x_fp32, long long ldx, int x_hs, co
                           cudaStream_t stream);
 /* y = tanh(u), fp32 in, ACT out */
 int llark_seq_tanh(const float* u, void* y, long long n, int act_fp32, cudaStream_t stream);
-/* C[off[e] .. off[e+1]) = A[same rows] @ B[e]^T, e < n_seg; B bf16 [n_seg, N, K]; seg_off_host on the host */
+/* C[off[e] .. off[e+1]) = A[same rows] @ B[e]^T, e < n_seg; B bf16 [n_seg, N, K]; seg_off_host on the host; epi:
+ * LLARK_EPI_NONE or LLARK_EPI_RELU2 */
 int llark_gemm_segments(const void* A, long long lda, const void* B, void* C, long long ldc, int c_fp32,
                         const int* seg_off_host, int n_seg, const int* seg_tiles_dev, int n_tiles, const int* seg_count_dev,
-                        int m_total, int N, int K, cudaStream_t stream);
+                        int m_total, int N, int K, int epi, cudaStream_t stream);
 /* routed mixture of experts (see csrc/seq_moe.cu) */
 int llark_seq_moe_route(const float* logits, long long ld, int* ids, float* wts, int n_tok, int n_exp, int n_groups,
                         int keep, int top, float scale, cudaStream_t stream);
@@ -446,6 +465,9 @@ int llark_seq_moe_route(const float* logits, long long ld, int* ids, float* wts,
  * weights = the chosen experts' plain scores * scale */
 int llark_seq_moe_route_bias(const float* logits, long long ld, const float* correction, int* ids, float* wts, int n_tok,
                              int n_exp, int n_groups, int keep, int top, float scale, cudaStream_t stream);
+/* the `top` largest logits of each row; weights = softmax over those logits */
+int llark_seq_moe_route_top(const float* logits, long long ld, int* ids, float* wts, int n_tok, int n_exp, int top,
+                            cudaStream_t stream);
 int llark_seq_moe_tile_rows(void);
 /* meta[0] = number of 64-row tiles; with tiles256: 256-row tiles for llark_gemm_segments, their number in meta[1];
  * experts >= n_real have no weights and get no tiles */
@@ -455,9 +477,9 @@ int llark_seq_moe_sort(const int* ids, int n_ent, int n_exp, int n_real, int* pe
 int llark_seq_moe_gather(const void* x, long long ldx, const int* perm, int top, void* xs, int n_ent, int C, int act_fp32,
                          cudaStream_t stream);
 int llark_seq_silu_mul(const void* gu, void* act, long long rows, int ff, int act_fp32, cudaStream_t stream);
-int llark_seq_moe_up(const void* x, long long ldx, const int* perm, int top, const void* w_gate_up, void* act,
-                     const int* tiles, const int* meta, int max_tiles, int n_ent, int ff, int K, int act_fp32,
-                     cudaStream_t stream);
+/* act[p] = silu(gate x) * (up x) with w [n, 2 * ff, K] (gated), or relu(w x)^2 with w [n, ff, K]; x = row perm[p] / top */
+int llark_seq_moe_up(const void* x, long long ldx, const int* perm, int top, const void* w, void* act, const int* tiles,
+                     const int* meta, int max_tiles, int n_ent, int ff, int K, int gated, int act_fp32, cudaStream_t stream);
 int llark_seq_moe_down(const void* act, const void* w_down, float* z, const int* tiles, const int* meta, int max_tiles,
                        int n_ent, int C, int ff, int act_fp32, cudaStream_t stream);
 

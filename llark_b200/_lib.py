@@ -27,6 +27,7 @@ SEQ_SYMBOLS = [
     "llark_seq_moe_down", "llark_seq_tanh", "llark_seq_moe_gather", "llark_seq_silu_mul",
     "llark_seq_qkv_headnorm", "llark_seq_skip_gate_group_norm", "llark_seq_post_norm", "llark_seq_glu_clamped",
     "llark_seq_logit_cap", "llark_seq_moe_route_bias", "llark_seq_qkv_rotary", "llark_seq_gated_norm_add",
+    "llark_seq_tanh_norm", "llark_seq_tanh_norm_add", "llark_seq_moe_route_top",
 ]
 # what libllark_serve.so (`make serve`: GEMM core + decode linears + the ops above) exports
 SERVE_SYMBOLS = SEQ_SYMBOLS + ["llark_last_cuda_error", "llark_init", "llark_gemm", "llark_gemm_ex", "llark_gemv",
@@ -56,7 +57,7 @@ class GemmEpilogue(ctypes.Structure):
                 ("i0", ctypes.c_int), ("i1", ctypes.c_int)]
 
 
-EPI_NONE, EPI_QUICK_GELU, EPI_ROPE, EPI_SWIGLU_BWD = 0, 1, 2, 3
+EPI_NONE, EPI_QUICK_GELU, EPI_ROPE, EPI_SWIGLU_BWD, EPI_RELU2, EPI_RELU_GLU = 0, 1, 2, 3, 5, 6
 
 
 class LlarkError(RuntimeError):
@@ -148,15 +149,18 @@ def lib():
             "llark_seq_add_rmsnorm": ([P, P, P, P, P, LL, I, F, I, P], I),
             "llark_seq_rmsnorm_rows": ([P, P, P, P, I, I, F, I, P], I),
             "llark_seq_relu2": ([P, P, LL, I, P], I),
-            "llark_linear_rows": ([P, LL, P, LL, P, LL, I, P, I, I, I, I, P], I),
-            "llark_linear_simt": ([P, LL, P, LL, P, LL, I, P, I, I, I, I, P], I),
+            "llark_linear_rows": ([P, LL, P, LL, P, LL, I, P, I, I, I, I, I, P], I),
+            "llark_linear_simt": ([P, LL, P, LL, P, LL, I, P, I, I, I, I, I, P], I),
             "llark_seq_qk_headnorm": ([P, LL, I, I, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, F, I, P], I),
             "llark_seq_qkv_headnorm": ([P, LL, I, I, I, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, F, I, I, P], I),
             "llark_seq_swa_attn": ([P, P, P, P, P, P, LL, P, P, P, P, P, P, I, I, I, I, I, I, I, I, P, I, I, F, P, I, I, P], I),
             "llark_seq_swa_attn_mma": ([P, P, P, P, P, P, LL, P, P, P, P, P, I, I, I, I, I, I, I, P, I, I, F, P, I, P], I),
-            "llark_seq_qkv_rotary": ([P, LL, I, I, I, P, P, P, I, I, P, I, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, I,
+            "llark_seq_qkv_rotary": ([P, LL, I, I, I, P, P, P, I, I, P, I, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, I, I,
                                       P], I),
             "llark_seq_gated_norm_add": ([P, P, P, LL, P, P, P, P, LL, I, F, I, P], I),
+            "llark_seq_tanh_norm": ([P, P, F, P, P, P, I, I, I, P], I),
+            "llark_seq_tanh_norm_add": ([P, P, P, P, P, I, F, P, P, F, P, P, P, P, LL, I, I, P], I),
+            "llark_seq_moe_route_top": ([P, LL, P, P, I, I, I, P], I),
             "llark_seq_kv_ring_write": ([P, P, P, P, P, P, P, P, I, I, I, I, I, P], I),
             "llark_seq_glr_scan": ([P, LL, I, I, I, P, P, P, P, P, P, P, P, P, I, I, I, I, P], I),
             "llark_seq_glr_combine": ([P, P, P, P, P, I, I, I, I, P], I),
@@ -180,9 +184,9 @@ def lib():
             "llark_seq_moe_sort": ([P, I, I, I, P, P, P, P, P, P, P], I),
             "llark_seq_moe_gather": ([P, LL, P, I, P, I, I, I, P], I),
             "llark_seq_silu_mul": ([P, P, LL, I, I, P], I),
-            "llark_seq_moe_up": ([P, LL, P, I, P, P, P, P, I, I, I, I, I, P], I),
+            "llark_seq_moe_up": ([P, LL, P, I, P, P, P, P, I, I, I, I, I, I, P], I),
             "llark_seq_moe_down": ([P, P, P, P, P, I, I, I, I, I, P], I),
-            "llark_gemm_segments": ([P, LL, P, P, LL, I, P, I, P, I, P, I, I, I, P], I),
+            "llark_gemm_segments": ([P, LL, P, P, LL, I, P, I, P, I, P, I, I, I, I, P], I),
             "llark_seq_tanh": ([P, P, LL, I, P], I),
         }
         for name, (argtypes, restype) in sig.items():

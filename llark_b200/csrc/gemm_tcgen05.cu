@@ -60,7 +60,8 @@ struct GemmParams {
                      // 2 = producer issues no TMA (MMA runs on stale smem: isolates the UMMA rate)
     // fused epilogue (LlarkGemmEpilogue): 0 none, 1 quick-GELU, 2 RoPE on the first epi_i1 columns (head_dim 128,
     // position = row % epi_i0, epi_a / epi_b = cos / sin bf16 [S,128]), 3 SwiGLU backward (epi_a = gu bf16 [M, epi_ld]:
-    // gate | up halves N apart; C receives dgate at column c and dup at column N + c)
+    // gate | up halves N apart; C receives dgate at column c and dup at column N + c), 5 squared ReLU, 6 gated ReLU (weight
+    // rows alternate gate, up: C column c = relu(acc column 2c) * acc column 2c + 1; C has N / 2 columns)
     int staged;      // 1 = staged (coalesced) epilogue, 0 = direct row-per-thread stores (see epilogue_dispatch)
     int group_m;     // m-blocks per rasterisation group (tile_coord): sized on the host so a group's A panel stays in L2
     int epi;
@@ -159,6 +160,25 @@ __device__ __forceinline__ void epilogue_store_chunk(const GemmParams& p, long l
             }
             st8_bf16(cptr, dg);
             st8_bf16(cptr + p.N, du);
+            continue;
+        } else if constexpr (EPI == 5) {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) {
+                const float r = fmaxf(f[e], 0.f);
+                f[e] = r * r;
+            }
+        } else if constexpr (EPI == 6) {
+            // gate / up columns alternate (N even, C bf16): four results per eight columns
+            __nv_bfloat16* cptr = reinterpret_cast<__nv_bfloat16*>(p.C) + row * p.ldc + (col >> 1);
+            float g[4];
+#pragma unroll
+            for (int e = 0; e < 4; ++e) g[e] = fmaxf(f[2 * e], 0.f) * f[2 * e + 1];
+            if (full8) {
+                *reinterpret_cast<uint2*>(cptr) = make_uint2(pack_bf16x2(g[0], g[1]), pack_bf16x2(g[2], g[3]));
+            } else {
+                for (int e = 0; e < 4; ++e)
+                    if (col + 2 * e < p.N) cptr[e] = __float2bfloat16_rn(g[e]);
+            }
             continue;
         }
         if (p.c_fp32) {
@@ -481,15 +501,17 @@ __device__ __forceinline__ void epi_staged_bf16(const GemmParams& p, long long r
 template <int EPI>
 __device__ __forceinline__ void epilogue_dispatch(const GemmParams& p, long long row0, long long m_end, int lane, int ncol0,
                                                   uint32_t taddr, float* stg) {
-    if ((EPI == 2 && ncol0 < p.epi_i1) || !p.staged) {
+    if ((EPI == 2 && ncol0 < p.epi_i1) || EPI == 5 || EPI == 6 || !p.staged) {
         const long long row = row0 + lane;
         epilogue_tile<EPI>(p, row, row < m_end, ncol0, taddr);
         return;
     }
-    if (p.c_fp32) {
-        if constexpr (EPI == 0 || EPI == 1) epi_staged_f32<EPI>(p, row0, ncol0, taddr, stg, lane);
-    } else {
-        epi_staged_bf16<EPI>(p, row0, ncol0, taddr, stg, lane);
+    if constexpr (EPI != 5 && EPI != 6) {  // these two have no staged form
+        if (p.c_fp32) {
+            if constexpr (EPI == 0 || EPI == 1) epi_staged_f32<EPI>(p, row0, ncol0, taddr, stg, lane);
+        } else {
+            epi_staged_bf16<EPI>(p, row0, ncol0, taddr, stg, lane);
+        }
     }
 }
 
@@ -1180,8 +1202,8 @@ extern "C" int llark_gemm_ex(const void* A, int a_mn_major, long long lda, const
     if (M <= 0 || N <= 0 || K <= 0 || !A || !B || !C) return LLARK_EINVAL;
     const bool segs = ep && ep->kind == LLARK_EPI_SEGMENTS;
     if (segs) {
-        // a = device tile list, i0 = its length, i1 = weight blocks stacked in B; plain output otherwise
-        if (!ep->a || ep->i0 <= 0 || ep->i1 <= 0 || a_mn_major || b_mn_major || in_fp32 || bias || R ||
+        // a = device tile list, i0 = its length, i1 = weight blocks stacked in B; ld = LLARK_EPI_NONE or LLARK_EPI_RELU2
+        if ((ep->ld != LLARK_EPI_NONE && ep->ld != LLARK_EPI_RELU2) || !ep->a || ep->i0 <= 0 || ep->i1 <= 0 || a_mn_major || b_mn_major || in_fp32 || bias || R ||
             !llark_gemm_get_mode())
             return LLARK_EINVAL;
     } else if (ep && ep->kind != LLARK_EPI_NONE) {
@@ -1200,6 +1222,12 @@ extern "C" int llark_gemm_ex(const void* A, int a_mn_major, long long lda, const
                 if (c_fp32 || bias || R || !ep->a || (N % 8) || (ep->ld % 8) || ep->ld < 2LL * N || ldc < 2LL * N ||
                     (reinterpret_cast<uintptr_t>(ep->a) & 15))
                     return LLARK_EINVAL;
+                break;
+            case LLARK_EPI_RELU2:
+                if (R || a_mn_major || b_mn_major || in_fp32) return LLARK_EINVAL;
+                break;
+            case LLARK_EPI_RELU_GLU:
+                if (R || a_mn_major || b_mn_major || in_fp32 || c_fp32 || (N % 2) || ldc < N / 2) return LLARK_EINVAL;
                 break;
             default:
                 return LLARK_EINVAL;
@@ -1268,7 +1296,7 @@ extern "C" int llark_gemm_ex(const void* A, int a_mn_major, long long lda, const
     }
     p.a_tma4 = a4 ? use4 : 0;
     p.b_tma4 = b4 ? use4 : 0;
-    p.epi = (ep && !segs) ? ep->kind : 0;
+    p.epi = !ep ? 0 : (segs ? (int)ep->ld : ep->kind);
     p.seg_tiles = segs ? static_cast<const int*>(ep->a) : nullptr;
     p.seg_count = segs ? static_cast<const int*>(ep->b) : nullptr;
     if (segs) p.num_m_blocks = ep->i0;
@@ -1335,6 +1363,12 @@ extern "C" int llark_gemm_ex(const void* A, int a_mn_major, long long lda, const
         if (p.epi == LLARK_EPI_SWIGLU_BWD && sel == 1 && !in_fp32)
             return two_cta ? launch2<0, 1, 0, 3>(ta, tb, p, max_ctas, stream)
                            : launch<0, 1, 0, 3>(ta, tb, p, max_ctas, stream);
+        if (p.epi == LLARK_EPI_RELU2 && sel == 0 && !in_fp32)
+            return two_cta ? launch2<0, 0, 0, 5>(ta, tb, p, max_ctas, stream)
+                           : launch<0, 0, 0, 5>(ta, tb, p, max_ctas, stream);
+        if (p.epi == LLARK_EPI_RELU_GLU && sel == 0 && !in_fp32)
+            return two_cta ? launch2<0, 0, 0, 6>(ta, tb, p, max_ctas, stream)
+                           : launch<0, 0, 0, 6>(ta, tb, p, max_ctas, stream);
         return LLARK_EINVAL;
     }
     if (two_cta) {
@@ -1377,18 +1411,20 @@ extern "C" void llark_gemm_clear_cache(void) {
 // first row, rows <= 256, covering every run) and the CTA-pair kernel this is ONE launch whose m-blocks follow the list;
 // n_tiles is the list's length or, with seg_count_dev (a device word holding the real length), an upper bound of it, so
 // that nothing about the runs has to be known on the host. Without a tile list: seg_off_host [n_seg + 1] gives the run
-// boundaries and every run is a launch of its own. bf16 operands, bf16 or fp32 output.
+// boundaries and every run is a launch of its own. bf16 operands, bf16 or fp32 output. epi: LLARK_EPI_NONE or
+// LLARK_EPI_RELU2.
 extern "C" int llark_gemm_segments(const void* A, long long lda, const void* B, void* C, long long ldc, int c_fp32,
                                    const int* seg_off_host, int n_seg, const int* seg_tiles_dev, int n_tiles,
-                                   const int* seg_count_dev, int m_total, int N, int K, cudaStream_t stream) {
-    if (!A || !B || !C || n_seg <= 0 || N <= 0 || K <= 0) return LLARK_EINVAL;
+                                   const int* seg_count_dev, int m_total, int N, int K, int epi, cudaStream_t stream) {
+    if (!A || !B || !C || n_seg <= 0 || N <= 0 || K <= 0 || (epi != LLARK_EPI_NONE && epi != LLARK_EPI_RELU2))
+        return LLARK_EINVAL;
     if (seg_tiles_dev && n_tiles > 0 && llark_gemm_get_mode()) {
         if (m_total <= 0) return LLARK_EINVAL;
         LlarkGemmEpilogue ep;
         ep.kind = LLARK_EPI_SEGMENTS;
         ep.a = seg_tiles_dev;
         ep.b = seg_count_dev;
-        ep.ld = 0;
+        ep.ld = epi;
         ep.i0 = n_tiles;
         ep.i1 = n_seg;
         return llark_gemm_ex(A, 0, lda, B, 0, K, C, ldc, c_fp32, nullptr, 0, nullptr, 0, m_total, N, K, 0, 0, &ep, stream);
@@ -1400,9 +1436,10 @@ extern "C" int llark_gemm_segments(const void* A, long long lda, const void* B, 
     for (int e = 0; e < n_seg; ++e) {
         const int r0 = seg_off_host[e], rows = seg_off_host[e + 1] - r0;
         if (rows <= 0) continue;
-        const int rc = llark_gemm(a + (long long)r0 * lda * 2, 0, lda, b + (long long)e * N * K * 2, 0, K,
-                                  c + (long long)r0 * ldc * (c_fp32 ? 4 : 2), ldc, c_fp32, nullptr, 0, nullptr, 0, rows, N, K,
-                                  0, 0, stream);
+        LlarkGemmEpilogue one = {epi, nullptr, nullptr, 0, 0, 0};
+        const int rc = llark_gemm_ex(a + (long long)r0 * lda * 2, 0, lda, b + (long long)e * N * K * 2, 0, K,
+                                     c + (long long)r0 * ldc * (c_fp32 ? 4 : 2), ldc, c_fp32, nullptr, 0, nullptr, 0, rows,
+                                     N, K, 0, 0, &one, stream);
         if (rc != LLARK_OK) return rc;
     }
     return LLARK_OK;

@@ -5,7 +5,9 @@
 //   llark_seq_qk_headnorm   per-head RMS norm of the q and k columns of a fused projection; the raw k is kept as well
 //                           (designs whose values are the un-normed keys); optionally writes the ring directly (decode)
 //   llark_seq_qkv_rotary    optional whole-projection RMS norm of q and k, rotary positions on q / k (halves or interleaved
-//                           pairs, partial head) and optionally on the values; optionally writes the rings (decode)
+//                           pairs, partial head) and optionally on the values, optional division of every rotated q / k head
+//                           by its own root mean square; queries alone where another layer's keys and values are used;
+//                           optionally writes the rings (decode)
 //   llark_seq_swa_attn      softmax attention over a sliding window (or the query's block of `chunk` positions; scores
 //                           optionally squashed by cap * tanh(s / cap); weighted value sums optionally turned back by the
 //                           query's position): keys of this step from the step's buffers, older
@@ -102,6 +104,9 @@ __global__ void qk_headnorm_kernel(const float* __restrict__ src, long long ld, 
 //            pair i = (i, i + n_rot/2) ("halves") or (2i, 2i+1) (qk_interleaved); the rest of the head passes
 //   v_freq [E / 2] (optional): every value head is rotated by its position the same way over all of E (v_interleaved);
 //            the attention kernels turn their weighted sums back by the query's position
+//   unit     every q and k head is divided by sqrt(mean over its D entries of the square + eps) after the rotation. A rotation
+//            leaves the sum of squares as it is, so the factor is taken from the row before it and applied in the same pass.
+//   G = 0    queries only (kn, vv, the rings and wk are not used)
 // Angles are float(position) * frequency, cos / sin in fp32. Results in T; with kring / vring the k / v rows also go to
 // ring entry position % cap of the token's slot (steps of one token per request).
 template <typename T>
@@ -112,7 +117,7 @@ __global__ void qkv_rotary_kernel(const float* __restrict__ src, long long ld, i
                                   T* __restrict__ kn, T* __restrict__ vv, T* __restrict__ kring, T* __restrict__ vring,
                                   const int* __restrict__ tok_seq, const int* __restrict__ cu,
                                   const int* __restrict__ pos0, const int* __restrict__ slot, int H, int G, int D, int E,
-                                  int cap, float eps) {
+                                  int cap, float eps, int unit) {
     extern __shared__ float cs[];  // cos | sin of the q / k pairs [2 * (n_rot / 2)], then of the value pairs [2 * (E / 2)]
     __shared__ float red[2][32];
     const int t = blockIdx.x;
@@ -120,6 +125,7 @@ __global__ void qkv_rotary_kernel(const float* __restrict__ src, long long ld, i
     const long long p = pos0[b] + (t - cu[b]);
     const int hq = n_rot >> 1, hv = v_freq ? (E >> 1) : 0;
     float* csv = cs + 2 * hq;
+    float* hr = csv + 2 * hv;  // [H + G] factors of the heads (unit)
     for (int i = threadIdx.x; i < hq; i += blockDim.x) sincosf((float)p * qk_freq[i], &cs[2 * i + 1], &cs[2 * i]);
     for (int i = threadIdx.x; i < hv; i += blockDim.x) sincosf((float)p * v_freq[i], &csv[2 * i + 1], &csv[2 * i]);
     const float* row = src + (long long)t * ld;
@@ -144,6 +150,14 @@ __global__ void qkv_rotary_kernel(const float* __restrict__ src, long long ld, i
         rq = 1.0f / sqrtf(sq / (float)(H * D) + eps);
         rk = 1.0f / sqrtf(sk / (float)(G * D) + eps);
     } else {
+        if (unit)
+            for (int hh = threadIdx.x >> 5; hh < H + G; hh += blockDim.x >> 5) {
+                const float* s = row + (hh < H ? q_off + hh * D : k_off + (hh - H) * D);
+                float ss = 0.f;
+                for (int c = threadIdx.x & 31; c < D; c += 32) ss = fmaf(s[c], s[c], ss);
+                ss = warp_sum(ss);
+                if ((threadIdx.x & 31) == 0) hr[hh] = 1.0f / sqrtf(ss / (float)D + eps);
+            }
         __syncthreads();
     }
     T *rk_row = nullptr, *rv_row = nullptr;
@@ -161,7 +175,7 @@ __global__ void qkv_rotary_kernel(const float* __restrict__ src, long long ld, i
         const int c0 = head * D;
         const float* s = row + (is_q ? q_off : k_off) + c0;
         const float* w = is_q ? wq : wk;
-        const float r = is_q ? rq : rk;
+        const float r = unit ? hr[hh] : (is_q ? rq : rk);
         T* o = is_q ? qn + (long long)t * H * D + c0 : kn + (long long)t * G * D + c0;
         T* o2 = (!is_q && rk_row) ? rk_row + c0 : nullptr;
         if (j < hq) {
@@ -291,7 +305,7 @@ __global__ void qkv_rotary4_kernel(const float* __restrict__ src, long long ld, 
                                    T* __restrict__ kn, T* __restrict__ vv, T* __restrict__ kring, T* __restrict__ vring,
                                    const int* __restrict__ tok_seq, const int* __restrict__ cu,
                                    const int* __restrict__ pos0, const int* __restrict__ slot, int H, int G, int D, int E,
-                                   int cap, float eps) {
+                                   int cap, float eps, int unit) {
     extern __shared__ float cs[];
     __shared__ float red[2][32];
     const int t = blockIdx.x;
@@ -299,6 +313,7 @@ __global__ void qkv_rotary4_kernel(const float* __restrict__ src, long long ld, 
     const long long p = pos0[b] + (t - cu[b]);
     const int hq = n_rot >> 1, hv = v_freq ? (E >> 1) : 0;
     float* csv = cs + 2 * hq;
+    float* hr = csv + 2 * hv;  // [H + G] factors of the heads (unit)
     for (int i = threadIdx.x; i < hq; i += blockDim.x) sincosf((float)p * qk_freq[i], &cs[2 * i + 1], &cs[2 * i]);
     for (int i = threadIdx.x; i < hv; i += blockDim.x) sincosf((float)p * v_freq[i], &csv[2 * i + 1], &csv[2 * i]);
     const float* row = src + (long long)t * ld;
@@ -329,6 +344,17 @@ __global__ void qkv_rotary4_kernel(const float* __restrict__ src, long long ld, 
         rq = 1.0f / sqrtf(sq / (float)(H * D) + eps);
         rk = 1.0f / sqrtf(sk / (float)(G * D) + eps);
     } else {
+        if (unit)
+            for (int hh = threadIdx.x >> 5; hh < H + G; hh += blockDim.x >> 5) {
+                const float4* s = reinterpret_cast<const float4*>(row + (hh < H ? q_off + hh * D : k_off + (hh - H) * D));
+                float ss = 0.f;
+                for (int c = threadIdx.x & 31; c < D >> 2; c += 32) {
+                    const float4 a = s[c];
+                    ss += a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w;
+                }
+                ss = warp_sum(ss);
+                if ((threadIdx.x & 31) == 0) hr[hh] = 1.0f / sqrtf(ss / (float)D + eps);
+            }
         __syncthreads();
     }
     T *rk_row = nullptr, *rv_row = nullptr;
@@ -347,7 +373,7 @@ __global__ void qkv_rotary4_kernel(const float* __restrict__ src, long long ld, 
             const bool is_q = hh < H;
             const int c0 = (is_q ? hh : hh - H) * D;
             const float* w = is_q ? wq : wk;
-            rotate_quads<T>(row + (is_q ? q_off : k_off) + c0, is_q ? rq : rk, w ? w + c0 : nullptr, cs, n_rot,
+            rotate_quads<T>(row + (is_q ? q_off : k_off) + c0, unit ? hr[hh] : (is_q ? rq : rk), w ? w + c0 : nullptr, cs, n_rot,
                             qk_interleaved, j, is_q ? qn + (long long)t * H * D + c0 : kn + (long long)t * G * D + c0,
                             (!is_q && rk_row) ? rk_row + c0 : (T*)nullptr);
         } else {
@@ -831,13 +857,14 @@ extern "C" int llark_seq_qkv_rotary(const float* src, long long ld, int q_off, i
                                     const float* wk, const float* qk_freq, int n_rot, int qk_interleaved,
                                     const float* v_freq, int v_interleaved, void* qn, void* kn, void* vv, void* kring,
                                     void* vring, const int* tok_seq, const int* cu, const int* pos0, const int* slot,
-                                    int n_tok, int H, int G, int D, int E, int cap, float eps, int act_fp32,
+                                    int n_tok, int H, int G, int D, int E, int cap, float eps, int unit, int act_fp32,
                                     cudaStream_t st) {
-    if (n_tok <= 0 || H <= 0 || G <= 0 || D <= 0 || E <= 0 || !src || !qn || !kn || !vv || !tok_seq || !cu || !pos0 ||
-        !slot || n_rot < 0 || (n_rot % 2) || n_rot > D || (n_rot && !qk_freq) || (!wq != !wk))
+    if (n_tok <= 0 || H <= 0 || G < 0 || D <= 0 || E <= 0 || !src || !qn || (G && (!kn || !vv)) || !tok_seq || !cu || !pos0 ||
+        !slot || n_rot < 0 || (n_rot % 2) || n_rot > D || (n_rot && !qk_freq) || (!wq != !wk) || (unit && wq) ||
+        (!G && (wq || kring || v_freq)))
         return LLARK_EINVAL;
     if (kring && (!vring || cap <= 0)) return LLARK_EINVAL;
-    const size_t smem = sizeof(float) * (size_t)(n_rot + (v_freq ? 2 * (E / 2) : 0));
+    const size_t smem = sizeof(float) * (size_t)(n_rot + (v_freq ? 2 * (E / 2) : 0) + (unit ? H + G : 0));
     if (smem > 48 * 1024) return LLARK_EINVAL;
     // Four entries per access when every head, zone and offset is a multiple of four entries (of eight for zones in halves)
     // and the rows start on 16-byte boundaries.
@@ -854,7 +881,7 @@ extern "C" int llark_seq_qkv_rotary(const float* src, long long ld, int q_off, i
 #define LLARK_ROTARY(KERNEL, T)                                                                                      \
     KERNEL<T><<<n_tok, threads, smem, st>>>(src, ld, q_off, k_off, v_off, wq, wk, qk_freq, n_rot, qk_interleaved, v_freq, \
                                             v_interleaved, (T*)qn, (T*)kn, (T*)vv, (T*)kring, (T*)vring, tok_seq, cu, pos0, \
-                                            slot, H, G, D, E, cap, eps)
+                                            slot, H, G, D, E, cap, eps, unit)
     if (quads) {
         if (act_fp32) LLARK_ROTARY(qkv_rotary4_kernel, float);
         else LLARK_ROTARY(qkv_rotary4_kernel, bf16_t);

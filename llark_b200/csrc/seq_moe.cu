@@ -1,5 +1,5 @@
-// Routed mixture of experts on the generation path: every token uses `top` of n small gated feed-forwards
-// down(silu(gate x) * (up x)). The router picks experts on the device, one kernel sorts the (token, choice) entries by
+// Routed mixture of experts on the generation path: every token uses `top` of n small feed-forwards
+// down(silu(gate x) * (up x)), or down(relu(up x)^2). The router picks experts on the device, one kernel sorts the (token, choice) entries by
 // expert and cuts each expert's run into row tiles, and two grouped GEMM launches walk that tile list (rows gathered
 // through the sort permutation). Large bf16 steps instead run every expert's rows through the tcgen05 GEMM core in its
 // rows-in-runs mode (llark_seq_moe_gather, llark_gemm_segments with the sort kernel's list of 256-row tiles and its
@@ -15,8 +15,10 @@
 //                           the best `keep` groups cannot be chosen; weights = the chosen experts' plain scores * scale,
 //                           not renormalised. Router outputs >= n_real are experts without weights that hand their input
 //                           through: the sort leaves them out of the tile lists, the residual kernel adds the input.
+//   llark_seq_moe_route_top   the `top` largest logits are chosen, weights = softmax over the chosen logits only
 //   llark_seq_moe_sort      entries -> perm (sorted by expert), pos_of (inverse), tiles (expert, first row, rows)
-//   llark_seq_moe_up        act[pos] = silu(W_gate,e x) * (W_up,e x)     x = the entry's token row
+//   llark_seq_moe_up        act[pos] = silu(W_gate,e x) * (W_up,e x), or relu(W_up,e x)^2 for experts without a gate;
+//                           x = the entry's token row
 //   llark_seq_moe_down      z[pos]   = W_down,e act[pos]                 fp32
 #include "common.cuh"
 
@@ -206,6 +208,52 @@ __global__ void route_bias_kernel(const float* __restrict__ logits, long long ld
     }
 }
 
+// Warp per token, logits in shared memory. The choice is made on the logits themselves (a softmax over all of them could
+// underflow and lose the order); ties go to the lower number.
+__global__ void route_top_kernel(const float* __restrict__ logits, long long ld, int* __restrict__ ids,
+                                 float* __restrict__ wts, int n_tok, int n_exp, int top) {
+    extern __shared__ float sm[];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+    const long long t = (long long)blockIdx.x * nw + warp;
+    if (t >= n_tok) return;
+    float* s = sm + (long long)warp * n_exp;  // logits; -inf once taken
+    for (int e = lane; e < n_exp; e += 32) s[e] = logits[t * ld + e];
+    __syncwarp();
+    float chosen = -INFINITY, first = 0.f;  // lane k keeps choice k (top <= 32)
+    int chosen_e = 0;
+    for (int k = 0; k < top; ++k) {
+        float bv = -INFINITY;
+        int be = 0x7fffffff;
+        for (int e = lane; e < n_exp; e += 32)
+            if (s[e] > bv) {
+                bv = s[e];
+                be = e;
+            }
+        for (int m = 16; m > 0; m >>= 1) {
+            const float ov = __shfl_xor_sync(0xffffffffu, bv, m);
+            const int oe = __shfl_xor_sync(0xffffffffu, be, m);
+            if (ov > bv || (ov == bv && oe < be)) {
+                bv = ov;
+                be = oe;
+            }
+        }
+        if (be >= n_exp) be = 0;  // no number compared greater (NaN logits): stay inside the tables
+        if (k == 0) first = bv;
+        if (lane == k) {
+            chosen = bv;
+            chosen_e = be;
+        }
+        if (lane == 0) s[be] = -INFINITY;
+        __syncwarp();
+    }
+    const float w = lane < top ? expf(chosen - first) : 0.f;
+    const float sum = warp_sum(w);
+    if (lane < top) {
+        ids[t * top + lane] = chosen_e;
+        wts[t * top + lane] = w / sum;
+    }
+}
+
 // ------------------------------------------------------------------------------------------------ sort by expert
 // One block. meta[0] = number of tiles; tiles[i] = (expert, first sorted row, rows). Experts >= n_real (no weights) keep
 // their place in the sorted order but get no tiles.
@@ -260,14 +308,18 @@ __global__ void sort_kernel(const int* __restrict__ ids, int n_ent, int n_exp, i
 }
 
 // ------------------------------------------------------------------------------------------------ grouped GEMMs
-// Block = one row tile of one expert x 64 output columns. DUAL: two weight matrices (gate rows, then up rows, of the
-// expert's [2 * N, K] block) and out = silu(a) * b; otherwise out = the product. Rows of A: gather ? perm[pos] / top : pos.
-template <typename T, typename TC, bool DUAL>
+// Block = one row tile of one expert x 64 output columns. MODE kSiluGlu: two weight matrices (gate rows, then up rows, of the
+// expert's [2 * N, K] block) and out = silu(a) * b; kRelu2: out = relu(product)^2; kPlain: the product. Rows of A:
+// gather ? perm[pos] / top : pos.
+enum { kPlain = 0, kSiluGlu = 1, kRelu2 = 2 };
+
+template <typename T, typename TC, int MODE>
 __global__ void __launch_bounds__(256)
 grouped_linear_kernel(const T* __restrict__ A, long long lda, const int* __restrict__ perm, int top,
                       const T* __restrict__ W, TC* __restrict__ Cm, long long ldc, const int* __restrict__ tiles,
                       const int* __restrict__ meta, int N, int K) {
     constexpr int BM = kTileRows, BN = 64, BK = 16;
+    constexpr bool DUAL = MODE == kSiluGlu;
     if ((int)blockIdx.y >= meta[0]) return;
     __shared__ float As[BK][BM + 4];
     __shared__ float Ws[DUAL ? 2 : 1][BK][BN + 4];
@@ -316,19 +368,24 @@ grouped_linear_kernel(const T* __restrict__ A, long long lda, const int* __restr
             if (m < nr && n < N) {
                 float y = acc[i][j];
                 if (DUAL) y = y * sigmoidf_(y) * acc2[i][j];
+                if (MODE == kRelu2) {
+                    y = fmaxf(y, 0.f);
+                    y *= y;
+                }
                 stf(Cm + (long long)(r0 + m) * ldc + n, y);
             }
         }
 }
 
-// Few rows per expert (decode): a warp owns one output column of one row tile and streams its weight row (DUAL: the gate
+// Few rows per expert (decode): a warp owns one output column of one row tile and streams its weight row (kSiluGlu: the gate
 // and the up row) once in 16-byte pieces; the tile's rows come from L1 / L2, eight at a time.
-template <typename T, typename TC, bool DUAL>
+template <typename T, typename TC, int MODE>
 __global__ void __launch_bounds__(256)
 grouped_rows_kernel(const T* __restrict__ A, long long lda, const int* __restrict__ perm, int top,
                     const T* __restrict__ W, TC* __restrict__ Cm, long long ldc, const int* __restrict__ tiles,
                     const int* __restrict__ meta, int N, int K, int vec_ok) {
     constexpr int MB = 8, VEC = 16 / (int)sizeof(T);
+    constexpr bool DUAL = MODE == kSiluGlu;
     if ((int)blockIdx.y >= meta[0]) return;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int n = blockIdx.x * (blockDim.x >> 5) + warp;
@@ -387,6 +444,10 @@ grouped_rows_kernel(const T* __restrict__ A, long long lda, const int* __restric
             if (DUAL) {
                 const float u = warp_sum(acc2[m]);
                 y = y * sigmoidf_(y) * u;
+            }
+            if (MODE == kRelu2) {
+                y = fmaxf(y, 0.f);
+                y *= y;
             }
             if (lane == 0 && m0 + m < nr) stf(Cm + (long long)(r0 + m0 + m) * ldc + n, y);
         }
@@ -456,6 +517,16 @@ extern "C" int llark_seq_moe_route_bias(const float* logits, long long ld, const
     return check_launch();
 }
 
+extern "C" int llark_seq_moe_route_top(const float* logits, long long ld, int* ids, float* wts, int n_tok, int n_exp, int top,
+                                       cudaStream_t st) {
+    if (n_tok <= 0 || n_exp <= 0 || top <= 0 || top > 32 || top > n_exp || !logits || !ids || !wts) return LLARK_EINVAL;
+    const int nw = 4;
+    const size_t smem = sizeof(float) * nw * (size_t)n_exp;
+    if (smem > 48 * 1024) return LLARK_EINVAL;
+    route_top_kernel<<<(n_tok + nw - 1) / nw, nw * 32, smem, st>>>(logits, ld, ids, wts, n_tok, n_exp, top);
+    return check_launch();
+}
+
 extern "C" int llark_seq_moe_tile_rows(void) { return kTileRows; }
 
 extern "C" int llark_seq_moe_sort(const int* ids, int n_ent, int n_exp, int n_real, int* perm, int* pos_of, int* tiles,
@@ -468,36 +539,34 @@ extern "C" int llark_seq_moe_sort(const int* ids, int n_ent, int n_exp, int n_re
     return check_launch();
 }
 
-extern "C" int llark_seq_moe_up(const void* x, long long ldx, const int* perm, int top, const void* w_gate_up, void* act,
-                                const int* tiles, const int* meta, int max_tiles, int n_ent, int ff, int K, int act_fp32,
-                                cudaStream_t st) {
-    if (max_tiles <= 0 || ff <= 0 || K <= 0 || top <= 0 || !x || !perm || !w_gate_up || !act || !tiles || !meta)
-        return LLARK_EINVAL;
+template <typename T, int MODE>
+static int launch_up(const void* x, long long ldx, const int* perm, int top, const void* w, void* act, const int* tiles,
+                     const int* meta, int max_tiles, int n_ent, int ff, int K, cudaStream_t st) {
     if (n_ent <= kRowsRouteMaxEntries) {  // a handful of rows per expert: stream the weights once
-        dim3 g2((ff + 7) / 8, max_tiles);
-        const int esz = act_fp32 ? 4 : 2, vec = 16 / esz;
+        const int vec = 16 / (int)sizeof(T);
         const int vec_ok = (K % vec == 0) && (ldx % vec == 0) &&
-                           (((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w_gate_up)) & 15) == 0);
-        if (act_fp32)
-            grouped_rows_kernel<float, float, true><<<g2, 256, 0, st>>>((const float*)x, ldx, perm, top,
-                                                                        (const float*)w_gate_up, (float*)act, ff, tiles,
-                                                                        meta, ff, K, vec_ok);
-        else
-            grouped_rows_kernel<bf16_t, bf16_t, true><<<g2, 256, 0, st>>>((const bf16_t*)x, ldx, perm, top,
-                                                                          (const bf16_t*)w_gate_up, (bf16_t*)act, ff,
-                                                                          tiles, meta, ff, K, vec_ok);
-        return check_launch();
+                           (((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w)) & 15) == 0);
+        grouped_rows_kernel<T, T, MODE><<<dim3((ff + 7) / 8, max_tiles), 256, 0, st>>>(
+            (const T*)x, ldx, perm, top, (const T*)w, (T*)act, ff, tiles, meta, ff, K, vec_ok);
+    } else {
+        grouped_linear_kernel<T, T, MODE><<<dim3((ff + 63) / 64, max_tiles), 256, 0, st>>>(
+            (const T*)x, ldx, perm, top, (const T*)w, (T*)act, ff, tiles, meta, ff, K);
     }
-    dim3 grid((ff + 63) / 64, max_tiles);
-    if (act_fp32)
-        grouped_linear_kernel<float, float, true><<<grid, 256, 0, st>>>((const float*)x, ldx, perm, top,
-                                                                        (const float*)w_gate_up, (float*)act, ff, tiles,
-                                                                        meta, ff, K);
-    else
-        grouped_linear_kernel<bf16_t, bf16_t, true><<<grid, 256, 0, st>>>((const bf16_t*)x, ldx, perm, top,
-                                                                          (const bf16_t*)w_gate_up, (bf16_t*)act, ff,
-                                                                          tiles, meta, ff, K);
     return check_launch();
+}
+
+// gated = 1: w holds gate rows, then up rows, [n, 2 * ff, K], act = silu(gate x) * (up x); gated = 0: w is [n, ff, K],
+// act = relu(w x)^2
+extern "C" int llark_seq_moe_up(const void* x, long long ldx, const int* perm, int top, const void* w, void* act,
+                                const int* tiles, const int* meta, int max_tiles, int n_ent, int ff, int K, int gated,
+                                int act_fp32, cudaStream_t st) {
+    if (max_tiles <= 0 || ff <= 0 || K <= 0 || top <= 0 || !x || !perm || !w || !act || !tiles || !meta)
+        return LLARK_EINVAL;
+    if (gated)
+        return act_fp32 ? launch_up<float, kSiluGlu>(x, ldx, perm, top, w, act, tiles, meta, max_tiles, n_ent, ff, K, st)
+                        : launch_up<bf16_t, kSiluGlu>(x, ldx, perm, top, w, act, tiles, meta, max_tiles, n_ent, ff, K, st);
+    return act_fp32 ? launch_up<float, kRelu2>(x, ldx, perm, top, w, act, tiles, meta, max_tiles, n_ent, ff, K, st)
+                    : launch_up<bf16_t, kRelu2>(x, ldx, perm, top, w, act, tiles, meta, max_tiles, n_ent, ff, K, st);
 }
 
 extern "C" int llark_seq_moe_down(const void* act, const void* w_down, float* z, const int* tiles, const int* meta,
@@ -509,21 +578,21 @@ extern "C" int llark_seq_moe_down(const void* act, const void* w_down, float* z,
         const int vec_ok = (ff % vec == 0) &&
                            (((reinterpret_cast<uintptr_t>(act) | reinterpret_cast<uintptr_t>(w_down)) & 15) == 0);
         if (act_fp32)
-            grouped_rows_kernel<float, float, false><<<g2, 256, 0, st>>>((const float*)act, ff, nullptr, 1,
+            grouped_rows_kernel<float, float, kPlain><<<g2, 256, 0, st>>>((const float*)act, ff, nullptr, 1,
                                                                          (const float*)w_down, z, C, tiles, meta, C, ff,
                                                                          vec_ok);
         else
-            grouped_rows_kernel<bf16_t, float, false><<<g2, 256, 0, st>>>((const bf16_t*)act, ff, nullptr, 1,
+            grouped_rows_kernel<bf16_t, float, kPlain><<<g2, 256, 0, st>>>((const bf16_t*)act, ff, nullptr, 1,
                                                                           (const bf16_t*)w_down, z, C, tiles, meta, C, ff,
                                                                           vec_ok);
         return check_launch();
     }
     dim3 grid((C + 63) / 64, max_tiles);
     if (act_fp32)
-        grouped_linear_kernel<float, float, false><<<grid, 256, 0, st>>>((const float*)act, ff, nullptr, 1,
+        grouped_linear_kernel<float, float, kPlain><<<grid, 256, 0, st>>>((const float*)act, ff, nullptr, 1,
                                                                          (const float*)w_down, z, C, tiles, meta, C, ff);
     else
-        grouped_linear_kernel<bf16_t, float, false><<<grid, 256, 0, st>>>((const bf16_t*)act, ff, nullptr, 1,
+        grouped_linear_kernel<bf16_t, float, kPlain><<<grid, 256, 0, st>>>((const bf16_t*)act, ff, nullptr, 1,
                                                                           (const bf16_t*)w_down, z, C, tiles, meta, C, ff);
     return check_launch();
 }

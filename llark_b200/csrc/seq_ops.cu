@@ -15,9 +15,16 @@
 //   llark_seq_gated_norm_add  x_out = x + rmsnorm(y * sigmoid(gate)) * w, optional ACT copy of rmsnorm(x_out) * w_next
 //   llark_seq_rmsnorm_rows  y[i] = rmsnorm(x[rows[i]]) * w -> ACT (final norm of the rows whose logits are wanted)
 //   llark_seq_relu2         y = relu(u)^2
-//   llark_linear_rows       C = A W^T (+ bias) for a handful of rows: weight-streaming, one or two output columns per warp
-//   llark_linear_simt       C = A W^T (+ bias), any shape, tiled SIMT with fp32 accumulation (the fp32 mode's GEMM and the
+//   llark_seq_tanh_norm     y = tanh(alpha * x) * w + b -> ACT: an element-wise squashing that stands where others have a norm
+//   llark_seq_tanh_norm_add x_out = x + tanh(alpha * f) * w + b with f = a sublayer's result and / or the weighted sum of the
+//                           outputs of a token's chosen experts; optional ACT copy of the next sublayer's tanh norm of x_out
+//   llark_linear_rows       C = act(A W^T (+ bias)) for a handful of rows: weight-streaming, one or two output columns per warp
+//   llark_linear_simt       C = act(A W^T (+ bias)), any shape, tiled SIMT with fp32 accumulation (the fp32 mode's GEMM and the
 //                           fallback for shapes the TMA descriptors of the tcgen05 core cannot take)
+//                           act: LLARK_ACT_NONE, LLARK_ACT_RELU2 (squared ReLU), LLARK_ACT_RELU_GLU (weight rows alternate gate,
+//                           up: output column c = relu(column 2c) * column 2c + 1)
+#include <initializer_list>
+
 #include "common.cuh"
 
 namespace llark {
@@ -389,6 +396,67 @@ __global__ void gated_norm_add_kernel(const float* __restrict__ x, const float* 
     for (int c = threadIdx.x; c < C; c += blockDim.x) stf(xa + c, rowbuf[c] * r2 * w_next[c]);  // each thread reads its own
 }
 
+// ------------------------------------------------------------------------------------------------ tanh norm
+// tanh(alpha * v) * w + b: no mean, no variance, so a row needs no reduction and its columns spread over blocks (grid: rows
+// x column blocks). tanhf: the squashing belongs to what is computed in full fp32.
+struct TanhNorm {
+    float alpha;
+    const float *w, *b;
+};
+__device__ __forceinline__ float tanh_norm1(float v, float alpha, float w, float b) { return fmaf(tanhf(alpha * v), w, b); }
+__device__ __forceinline__ float4 tanh_norm4(float4 v, const TanhNorm& n, int c4) {
+    const float4 w = __ldg(reinterpret_cast<const float4*>(n.w) + c4), b = __ldg(reinterpret_cast<const float4*>(n.b) + c4);
+    return make_float4(tanh_norm1(v.x, n.alpha, w.x, b.x), tanh_norm1(v.y, n.alpha, w.y, b.y),
+                       tanh_norm1(v.z, n.alpha, w.z, b.z), tanh_norm1(v.w, n.alpha, w.w, b.w));
+}
+
+template <typename T, bool VEC>
+__global__ void tanh_norm_kernel(const float* __restrict__ x, const int* __restrict__ rows, TanhNorm n, T* __restrict__ out,
+                                 int C) {
+    const long long r = blockIdx.x, src = rows ? rows[r] : r;
+    const int i = blockIdx.y * blockDim.x + threadIdx.x;
+    if (VEC) {
+        if (i >= (C >> 2)) return;
+        const float4 v = tanh_norm4(reinterpret_cast<const float4*>(x + src * C)[i], n, i);
+        st4(out + r * C + 4 * i, v.x, v.y, v.z, v.w);
+    } else if (i < C) {
+        stf(out + r * C + i, tanh_norm1(x[src * C + i], n.alpha, n.w[i], n.b[i]));
+    }
+}
+
+// f = y (optional) + sum over the token's `top` choices of wts[t, k] * z[pos_of[t, k]], the choices in order.
+template <typename T, bool VEC>
+__global__ void tanh_norm_add_kernel(const float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ z,
+                                     const int* __restrict__ pos_of, const float* __restrict__ wts, int top, TanhNorm post,
+                                     TanhNorm next, float* __restrict__ x_out, T* __restrict__ x_act, int C) {
+    const long long t = blockIdx.x;
+    const int i = blockIdx.y * blockDim.x + threadIdx.x;
+    if (VEC) {
+        if (i >= (C >> 2)) return;
+        const float4 xv = reinterpret_cast<const float4*>(x + t * C)[i];
+        float4 f = y ? reinterpret_cast<const float4*>(y + t * C)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+        for (int k = 0; k < top; ++k) {
+            const float wt = __ldg(wts + t * top + k);
+            const float4 e = __ldg(reinterpret_cast<const float4*>(z + (long long)__ldg(pos_of + t * top + k) * C) + i);
+            f = make_float4(fmaf(wt, e.x, f.x), fmaf(wt, e.y, f.y), fmaf(wt, e.z, f.z), fmaf(wt, e.w, f.w));
+        }
+        const float4 d = tanh_norm4(f, post, i);
+        const float4 o = make_float4(xv.x + d.x, xv.y + d.y, xv.z + d.z, xv.w + d.w);
+        reinterpret_cast<float4*>(x_out + t * C)[i] = o;
+        if (x_act) {
+            const float4 h = tanh_norm4(o, next, i);
+            st4(x_act + t * C + 4 * i, h.x, h.y, h.z, h.w);
+        }
+    } else if (i < C) {
+        float f = y ? y[t * C + i] : 0.f;
+        for (int k = 0; k < top; ++k) f = fmaf(wts[t * top + k], z[(long long)pos_of[t * top + k] * C + i], f);
+        const float o = x[t * C + i] + tanh_norm1(f, post.alpha, post.w[i], post.b[i]);
+        x_out[t * C + i] = o;
+        if (x_act) stf(x_act + t * C + i, tanh_norm1(o, next.alpha, next.w[i], next.b[i]));
+    }
+}
+
 template <typename T>
 __global__ void rmsnorm_rows_kernel(const float* __restrict__ x, const int* __restrict__ rows, const float* __restrict__ w,
                                     T* __restrict__ out, int C, float eps) {
@@ -422,7 +490,7 @@ __global__ void tanh_kernel(const float* __restrict__ u, T* __restrict__ y, long
 template <typename T, typename TC, int MB, int NC>
 __global__ void __launch_bounds__(256)
 linear_rows_kernel(const T* __restrict__ A, long long lda, const T* __restrict__ W, long long ldw, TC* __restrict__ Cm,
-                   long long ldc, const float* __restrict__ bias, int M, int N, int K, int vec_ok) {
+                   long long ldc, const float* __restrict__ bias, int M, int N, int K, int vec_ok, int act) {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const long long n0 = ((long long)blockIdx.x * (blockDim.x >> 5) + warp) * NC;
     const int m0 = blockIdx.y * MB;
@@ -468,13 +536,28 @@ linear_rows_kernel(const T* __restrict__ A, long long lda, const T* __restrict__
                 if (m0 + m < M) acc[m][c] = fmaf(ldf(A + (long long)(m0 + m) * lda + k), wv, acc[m][c]);
         }
     }
+    if (NC == 2 && act == LLARK_ACT_RELU_GLU) {  // the warp's two columns are a gate and its up column (N is even)
+#pragma unroll
+        for (int m = 0; m < MB; ++m) {
+            const float g = warp_sum(acc[m][0]) + (bias ? bias[n0] : 0.f);
+            const float u = warp_sum(acc[m][NC - 1]) + (bias ? bias[n0 + 1] : 0.f);
+            if (lane == 0 && m0 + m < M) stf(Cm + (long long)(m0 + m) * ldc + (n0 >> 1), fmaxf(g, 0.f) * u);
+        }
+        return;
+    }
 #pragma unroll
     for (int m = 0; m < MB; ++m)
 #pragma unroll
         for (int c = 0; c < NC; ++c) {
-            const float s = warp_sum(acc[m][c]);
-            if (lane == 0 && m0 + m < M && n0 + c < N)
-                stf(Cm + (long long)(m0 + m) * ldc + n0 + c, s + (bias ? bias[n0 + c] : 0.f));
+            float s = warp_sum(acc[m][c]);
+            if (lane == 0 && m0 + m < M && n0 + c < N) {
+                s += bias ? bias[n0 + c] : 0.f;
+                if (act == LLARK_ACT_RELU2) {
+                    s = fmaxf(s, 0.f);
+                    s *= s;
+                }
+                stf(Cm + (long long)(m0 + m) * ldc + n0 + c, s);
+            }
         }
 }
 
@@ -482,7 +565,7 @@ linear_rows_kernel(const T* __restrict__ A, long long lda, const T* __restrict__
 template <typename T, typename TC, typename TW = T>
 __global__ void __launch_bounds__(256)
 linear_simt_kernel(const T* __restrict__ A, long long lda, const TW* __restrict__ W, long long ldw, TC* __restrict__ Cm,
-                   long long ldc, const float* __restrict__ bias, int M, int N, int K) {
+                   long long ldc, const float* __restrict__ bias, int M, int N, int K, int act) {
     constexpr int BM = 64, BN = 64, BK = 16;
     __shared__ float As[BK][BM + 4];
     __shared__ float Ws[BK][BN + 4];
@@ -515,7 +598,19 @@ linear_simt_kernel(const T* __restrict__ A, long long lda, const TW* __restrict_
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int m = m0 + ty * 4 + i, n = n0 + tx * 4 + j;
-            if (m < M && n < N) stf(Cm + (long long)m * ldc + n, acc[i][j] + (bias ? bias[n] : 0.f));
+            if (m >= M || n >= N) continue;
+            float s = acc[i][j] + (bias ? bias[n] : 0.f);
+            if (act == LLARK_ACT_RELU_GLU) {  // n even: the gate; its up column is the next one of this thread (N is even)
+                if (j & 1) continue;
+                const float u = acc[i][(j + 1) & 3] + (bias ? bias[n + 1] : 0.f);
+                stf(Cm + (long long)m * ldc + (n >> 1), fmaxf(s, 0.f) * u);
+                continue;
+            }
+            if (act == LLARK_ACT_RELU2) {
+                s = fmaxf(s, 0.f);
+                s *= s;
+            }
+            stf(Cm + (long long)m * ldc + n, s);
         }
 }
 
@@ -791,6 +886,11 @@ __global__ void linear_rows_w32_kernel(const TA* __restrict__ A, long long lda, 
     }
 }
 
+static bool bad_act(int act, int N) {
+    return act < LLARK_ACT_NONE || act > LLARK_ACT_RELU_GLU || (act == LLARK_ACT_RELU_GLU && (N % 2));
+}
+static long long out_cols(int act, int N) { return act == LLARK_ACT_RELU_GLU ? N / 2 : N; }
+
 static int norm_threads(int C) {
     int t = 32;
     while (t < C / 4 && t < 512) t <<= 1;
@@ -924,6 +1024,63 @@ extern "C" int llark_seq_gated_norm_add(const float* x, const float* y, const fl
     return check_launch();
 }
 
+static bool aligned16(std::initializer_list<const void*> ps) {
+    for (const void* p : ps)
+        if (reinterpret_cast<uintptr_t>(p) & 15) return false;
+    return true;
+}
+// threads and column blocks of a row of C columns (VEC: four columns per thread)
+static void tanh_norm_shape(int C, bool vec, int& threads, unsigned& gy) {
+    const int items = vec ? C / 4 : C;
+    threads = items >= 256 ? 256 : (items + 31) / 32 * 32;
+    gy = (unsigned)((items + threads - 1) / threads);
+}
+
+extern "C" int llark_seq_tanh_norm(const float* x, const int* rows, float alpha, const float* w, const float* b, void* out,
+                                   int n_rows, int C, int out_fp32, cudaStream_t st) {
+    if (n_rows <= 0 || C <= 0 || !x || !w || !b || !out) return LLARK_EINVAL;
+    const bool vec = C % 4 == 0 && aligned16({x, w, b, out});
+    const TanhNorm n{alpha, w, b};
+    int threads;
+    unsigned gy;
+    tanh_norm_shape(C, vec, threads, gy);
+    const dim3 grid((unsigned)n_rows, gy);
+    if (out_fp32) {
+        if (vec) tanh_norm_kernel<float, true><<<grid, threads, 0, st>>>(x, rows, n, (float*)out, C);
+        else tanh_norm_kernel<float, false><<<grid, threads, 0, st>>>(x, rows, n, (float*)out, C);
+    } else {
+        if (vec) tanh_norm_kernel<bf16_t, true><<<grid, threads, 0, st>>>(x, rows, n, (bf16_t*)out, C);
+        else tanh_norm_kernel<bf16_t, false><<<grid, threads, 0, st>>>(x, rows, n, (bf16_t*)out, C);
+    }
+    return check_launch();
+}
+
+extern "C" int llark_seq_tanh_norm_add(const float* x, const float* y, const float* z, const int* pos_of, const float* wts,
+                                       int top, float alpha, const float* w, const float* b, float next_alpha,
+                                       const float* next_w, const float* next_b, float* x_out, void* x_act, long long rows,
+                                       int C, int act_fp32, cudaStream_t st) {
+    if (rows <= 0 || C <= 0 || top < 0 || !x || !w || !b || !x_out || (!y && top == 0) ||
+        (top > 0 && (!z || !pos_of || !wts)) || (x_act && (!next_w || !next_b)))
+        return LLARK_EINVAL;
+    const bool vec = C % 4 == 0 && aligned16({x, y, z, w, b, next_w, next_b, x_out, x_act});
+    const TanhNorm post{alpha, w, b}, next{next_alpha, next_w, next_b};
+    int threads;
+    unsigned gy;
+    tanh_norm_shape(C, vec, threads, gy);
+    const dim3 grid((unsigned)rows, gy);
+#define LLARK_TNA(T, VEC) \
+    tanh_norm_add_kernel<T, VEC><<<grid, threads, 0, st>>>(x, y, z, pos_of, wts, top, post, next, x_out, (T*)x_act, C)
+    if (act_fp32) {
+        if (vec) LLARK_TNA(float, true);
+        else LLARK_TNA(float, false);
+    } else {
+        if (vec) LLARK_TNA(bf16_t, true);
+        else LLARK_TNA(bf16_t, false);
+    }
+#undef LLARK_TNA
+    return check_launch();
+}
+
 extern "C" int llark_seq_rmsnorm_rows(const float* x, const int* rows, const float* w, void* out, int n_rows, int C,
                                       float eps, int act_fp32, cudaStream_t st) {
     if (n_rows <= 0 || C <= 0 || !x || !w || !out) return LLARK_EINVAL;
@@ -947,18 +1104,18 @@ extern "C" int llark_seq_relu2(const void* u, void* y, long long n, int act_fp32
 
 template <typename T, typename TC>
 static void launch_rows(const void* A, long long lda, const void* W, long long ldw, void* C, long long ldc,
-                        const float* bias, int M, int N, int K, cudaStream_t st) {
+                        const float* bias, int M, int N, int K, int act, cudaStream_t st) {
     const int vec = 16 / (int)sizeof(T);
     const int vec_ok = (K % vec == 0) && (lda % vec == 0) && (ldw % vec == 0) &&
                        (((reinterpret_cast<uintptr_t>(A) | reinterpret_cast<uintptr_t>(W)) & 15) == 0);
     const int warps = 8;
     // two columns per warp once that still leaves several warps per SM (148 SMs); one for narrow outputs
-    const bool two = (long long)N >= 2LL * warps * 148 * 2;
+    const bool two = (long long)N >= 2LL * warps * 148 * 2 || act == LLARK_ACT_RELU_GLU;  // (a gate and its up column)
     const int nc = two ? 2 : 1;
     const unsigned gx = (unsigned)((N + warps * nc - 1) / (warps * nc));
 #define LLARK_ROWS(MB_, NC_)                                                                                            \
     linear_rows_kernel<T, TC, MB_, NC_><<<dim3(gx, (M + MB_ - 1) / MB_), warps * 32, 0, st>>>(                          \
-        (const T*)A, lda, (const T*)W, ldw, (TC*)C, ldc, bias, M, N, K, vec_ok)
+        (const T*)A, lda, (const T*)W, ldw, (TC*)C, ldc, bias, M, N, K, vec_ok, act)
     if (M <= 2) {
         if (two) LLARK_ROWS(2, 2);
         else LLARK_ROWS(2, 1);
@@ -970,32 +1127,36 @@ static void launch_rows(const void* A, long long lda, const void* W, long long l
 }
 
 extern "C" int llark_linear_rows(const void* A, long long lda, const void* W, long long ldw, void* C, long long ldc,
-                                 int c_fp32, const float* bias, int M, int N, int K, int in_fp32, cudaStream_t st) {
-    if (M <= 0 || N <= 0 || K <= 0 || !A || !W || !C || lda < K || ldw < K || ldc < N) return LLARK_EINVAL;
+                                 int c_fp32, const float* bias, int M, int N, int K, int in_fp32, int act,
+                                 cudaStream_t st) {
+    if (M <= 0 || N <= 0 || K <= 0 || !A || !W || !C || lda < K || ldw < K || bad_act(act, N) || ldc < out_cols(act, N))
+        return LLARK_EINVAL;
     if (in_fp32 && !c_fp32) return LLARK_EINVAL;
     if (in_fp32)
-        launch_rows<float, float>(A, lda, W, ldw, C, ldc, bias, M, N, K, st);
+        launch_rows<float, float>(A, lda, W, ldw, C, ldc, bias, M, N, K, act, st);
     else if (c_fp32)
-        launch_rows<bf16_t, float>(A, lda, W, ldw, C, ldc, bias, M, N, K, st);
+        launch_rows<bf16_t, float>(A, lda, W, ldw, C, ldc, bias, M, N, K, act, st);
     else
-        launch_rows<bf16_t, bf16_t>(A, lda, W, ldw, C, ldc, bias, M, N, K, st);
+        launch_rows<bf16_t, bf16_t>(A, lda, W, ldw, C, ldc, bias, M, N, K, act, st);
     return check_launch();
 }
 
 extern "C" int llark_linear_simt(const void* A, long long lda, const void* W, long long ldw, void* C, long long ldc,
-                                 int c_fp32, const float* bias, int M, int N, int K, int in_fp32, cudaStream_t st) {
-    if (M <= 0 || N <= 0 || K <= 0 || !A || !W || !C || lda < K || ldw < K || ldc < N) return LLARK_EINVAL;
+                                 int c_fp32, const float* bias, int M, int N, int K, int in_fp32, int act,
+                                 cudaStream_t st) {
+    if (M <= 0 || N <= 0 || K <= 0 || !A || !W || !C || lda < K || ldw < K || bad_act(act, N) || ldc < out_cols(act, N))
+        return LLARK_EINVAL;
     if (in_fp32 && !c_fp32) return LLARK_EINVAL;
     dim3 grid((N + 63) / 64, (M + 63) / 64);
     if (in_fp32)
         linear_simt_kernel<float, float><<<grid, 256, 0, st>>>((const float*)A, lda, (const float*)W, ldw, (float*)C, ldc,
-                                                               bias, M, N, K);
+                                                               bias, M, N, K, act);
     else if (c_fp32)
         linear_simt_kernel<bf16_t, float><<<grid, 256, 0, st>>>((const bf16_t*)A, lda, (const bf16_t*)W, ldw, (float*)C,
-                                                                ldc, bias, M, N, K);
+                                                                ldc, bias, M, N, K, act);
     else
         linear_simt_kernel<bf16_t, bf16_t><<<grid, 256, 0, st>>>((const bf16_t*)A, lda, (const bf16_t*)W, ldw, (bf16_t*)C,
-                                                                 ldc, bias, M, N, K);
+                                                                 ldc, bias, M, N, K, act);
     return check_launch();
 }
 
@@ -1013,10 +1174,11 @@ extern "C" int llark_linear_simt_w32(const void* A, long long lda, const float* 
     }
     dim3 grid((N + 63) / 64, (M + 63) / 64);
     if (in_fp32)
-        linear_simt_kernel<float, float, float><<<grid, 256, 0, st>>>((const float*)A, lda, W, ldw, C, ldc, bias, M, N, K);
+        linear_simt_kernel<float, float, float><<<grid, 256, 0, st>>>((const float*)A, lda, W, ldw, C, ldc, bias, M, N, K,
+                                                                     LLARK_ACT_NONE);
     else
         linear_simt_kernel<bf16_t, float, float><<<grid, 256, 0, st>>>((const bf16_t*)A, lda, W, ldw, C, ldc, bias, M, N,
-                                                                      K);
+                                                                      K, LLARK_ACT_NONE);
     return check_launch();
 }
 

@@ -30,6 +30,9 @@ the same packed weights and stores of its own.
     "moe_softmax_bias"  BiasedSoftmaxExperts  softmax router whose choice is made on score + a stored correction (groups
                                         ranked by their best), weights = plain scores, and trailing experts without
                                         weights that hand their input through
+    "relu_glu"   ReluGluFF              down(relu(gate x) * (up x)), one GEMM with the product in its epilogue
+    "moe_top_softmax"  TopSoftmaxExperts  biased router, the largest logits are chosen, weights = softmax over those logits;
+                                        experts (and an optional shared expert that every token uses) are relu(up x)^2 units
 
     "rotary_attention"  RotaryAttention   grouped-query softmax attention with rotary positions on q and k (halves or
                                         interleaved pairs, part of the head, optionally rescaled frequencies), optional
@@ -38,11 +41,19 @@ the same packed weights and stores of its own.
     "rotary_attention_vrot"  ValueRotaryAttention   the same with biased projections, an RMS norm over the WHOLE q and k
                                         projections, interleaved pairs, values that are stored rotated by their own position
                                         (the head outputs are turned back by the query's) and a 1 in every softmax denominator
+    "rotary_attention_unit"  UnitRotaryAttention   rotary_attention with biased projections, every rotated q / k head divided by
+                                        its own root mean square, no gate; `kv_from` in its configuration: the layer has no
+                                        keys and values of its own and reads those of an earlier layer (its stores, and what
+                                        the current step brought)
     "latent_attention_causal"  LatentCausalAttention   latent attention over everything before (per-position store), rotary
                                         halves, one gate per head
 
 Mixers that take `side=(matrix name, bias name)` compute that projection of their input inside their fused input GEMM and
 leave it in `self.side` (fp32 view) after forward(): a layer's gate on the sublayer's result reads the same input.
+
+Mixers that can read another layer's keys and values take `lender`, that layer's mixer object on the same cache. A feed-forward's
+`terms(x_act)` names the parts of its result (y, and / or the chosen experts' rows z with pos_of and wts) for residual kernels
+that add them up themselves.
 
 A mixer's `branches(x_act, st, cache)` returns ([(output fp32, norm weight or None), ...], scale): what the layer's residual
 kernel adds up (each output first RMS-normed with its weight when there is one). The default is the one output of forward().
@@ -175,8 +186,31 @@ class ReluSquaredFF:
         self.w, self.act = weights, act
 
     def forward(self, x_act):
-        u = ops.linear(x_act, self.w.w_up, out_dtype=self.act)
-        return ops.linear(ops.seq_relu2(u), self.w.w_down, out_dtype=F32)
+        return ops.linear(ops.linear(x_act, self.w.w_up, out_dtype=self.act, act="relu2"), self.w.w_down, out_dtype=F32)
+
+    def terms(self, x_act):
+        return {"y": self.forward(x_act)}
+
+
+class ReluGluFFWeights:
+    def __init__(self, w, pfx, spec, width, dev, act):
+        F = int(spec["ff"])
+        gate, up, self.w_down = (_mat(w, pfx + n, dev, act) for n in ("gate", "up", "down"))
+        _expect(pfx, ((gate, (F, width)), (up, (F, width)), (self.w_down, (width, F))))
+        self.w_gu = torch.stack([gate, up], dim=1).reshape(2 * F, width).contiguous()  # rows alternate gate, up
+
+
+class ReluGluFF:
+    Weights = ReluGluFFWeights
+
+    def __init__(self, weights, act):
+        self.w, self.act = weights, act
+
+    def forward(self, x_act):
+        return ops.linear(ops.linear(x_act, self.w.w_gu, out_dtype=self.act, act="relu_glu"), self.w.w_down, out_dtype=F32)
+
+    def terms(self, x_act):
+        return {"y": self.forward(x_act)}
 
 
 WINDOW_ALL = 1 << 30  # "window" of an attention that sees every earlier position
@@ -513,6 +547,8 @@ class RotaryAttentionWeights:
     rotate_values = False     # values are stored rotated by their position over all of vdim; outputs are turned back
     plus_one = False          # a 1 joins every softmax denominator (a key of score 0 without a value)
     mask_kind = "chunk"       # what mask.size means: "chunk" = blocks of positions counted from 0, "window" = sliding
+    gated = True              # element-wise sigmoid gate `g` in front of the output matrix
+    unit_heads = False        # every rotated q / k head is divided by its root mean square (no weight)
 
     def __init__(self, w, pfx, spec, width, dev, act, side=None):
         H, D = int(spec["heads"]), int(spec["dim"])
@@ -520,6 +556,7 @@ class RotaryAttentionWeights:
         if H % G:
             raise ValueError(f"{pfx}: heads must be a multiple of kv_heads")
         self.H, self.G, self.D, self.E = H, G, D, E
+        self.kv_from = spec.get("kv_from")  # number of the layer whose keys and values this one reads (None: its own)
         mask = spec.get("mask") or {}
         self.span = int(mask["size"]) if mask.get("size") else None  # None: every earlier position
         if self.span is not None and self.span <= 0:
@@ -541,11 +578,11 @@ class RotaryAttentionWeights:
             if E % 2:
                 raise ValueError(f"{pfx}: rotated values need an even vdim")
             self.v_freq = rotary_frequencies(E, rot["base"])[0].to(device=dev, dtype=F32).contiguous()
-        # one projection for (side |) q | k | v | gate
-        names = ("q", "k", "v", "g")
+        # one projection for (side |) q | k | v | gate, or the parts of it that the layer has
+        rows = {"q": H * D, "k": G * D, "v": G * E, "g": H * E}
+        names = [n for n in rows if (n != "g" or self.gated) and (n not in "kv" or self.kv_from is None)]
         parts = [_mat(w, pfx + n, dev, act) for n in names]
-        _expect(pfx, ((parts[0], (H * D, width)), (parts[1], (G * D, width)), (parts[2], (G * E, width)),
-                      (parts[3], (H * E, width))))
+        _expect(pfx, [(m, (rows[n], width)) for n, m in zip(names, parts)])
         bias = [(_vec(w, pfx + n + ".b", dev) if self.biases and n != "g" else torch.zeros(m.shape[0], device=dev, dtype=F32))
                 for n, m in zip(names, parts)]
         self.side_n = 0
@@ -554,9 +591,11 @@ class RotaryAttentionWeights:
             self.side_n = parts[0].shape[0]
             _expect(pfx, ((parts[0], (self.side_n, width)),))
             bias.insert(0, _vec(w, side[1], dev) if side[1] is not None else torch.zeros(self.side_n, device=dev, dtype=F32))
-        self.q_off = self.side_n
-        self.k_off, self.v_off, self.g_off = self.q_off + H * D, self.q_off + (H + G) * D, self.q_off + (H + G) * D + G * E
-        self.n_in = self.g_off + H * E
+        at, offs = self.side_n, {}
+        for n in rows:  # a part that is not there takes no columns
+            offs[n] = at
+            at += rows[n] if n in names else 0
+        self.q_off, self.k_off, self.v_off, self.g_off, self.n_in = offs["q"], offs["k"], offs["v"], offs["g"], at
         self.w_in = _pad_rows(torch.cat(parts))
         self.b_in = None
         if self.biases or (side is not None and side[1] is not None):
@@ -575,11 +614,21 @@ class RotaryAttentionWeights:
 class RotaryAttention(_OneBranch):
     Weights = RotaryAttentionWeights
 
-    def __init__(self, weights, cache, eps, act, max_positions=None):
+    def __init__(self, weights, cache, eps, act, max_positions=None, lender=None):
         self.w, self.eps, self.act = weights, float(eps), act
         self.side = None
+        self.lender, self.lends, self.step_kv = lender, False, None
         w = weights
-        if w.span is None:  # one entry per position, grown by the cache
+        if (w.kv_from is None) != (lender is None):
+            raise ValueError("a mixer with kv_from, and no other, needs the mixer it reads keys and values from")
+        if lender is not None:
+            o = lender.w
+            if lender.lender is not None or lender.ring is not None:
+                raise ValueError("keys and values are read from a layer that has its own, kept for every position")
+            if (o.G, o.D, o.E) != (w.G, w.D, w.E):
+                raise ValueError("kv_heads, dim and vdim of a layer and of the one it reads keys and values from must agree")
+            lender.lends, self.ring, self.h_k, self.h_v = True, None, lender.h_k, lender.h_v
+        elif w.span is None:  # one entry per position, grown by the cache
             self.ring = None
             self.h_k = cache.add_store((w.G * w.D,), act, zero_on_alloc=False, per_position=True)
             self.h_v = cache.add_store((w.G * w.E,), act, zero_on_alloc=False, per_position=True)
@@ -595,18 +644,29 @@ class RotaryAttention(_OneBranch):
         kring, vring = cache.view(self.h_k), cache.view(self.h_v)
         cap = self.ring if self.ring is not None else cache.positions
         single = st.max_len == 1
-        q, k, v = ops.seq_qkv_rotary(pin, w.q_off, w.k_off, w.v_off, w.H, w.G, w.D, w.E, self.eps, self.act, st,
+        own = self.lender is None
+        write = single and own  # one token per request: its keys and values go straight into the stores
+        q, k, v = ops.seq_qkv_rotary(pin, w.q_off, w.k_off, w.v_off, w.H, w.G if own else 0, w.D, w.E, self.eps, self.act, st,
                                      wq=w.q_norm, wk=w.k_norm, qk_freq=w.qk_freq, qk_interleaved=w.interleaved,
-                                     v_freq=w.v_freq, v_interleaved=w.interleaved,
-                                     kring=kring if single else None, vring=vring if single else None, cap=cap)
+                                     v_freq=w.v_freq if own else None, v_interleaved=w.interleaved,
+                                     kring=kring if write else None, vring=vring if write else None, cap=cap,
+                                     unit=w.unit_heads)
+        if not own and not single:  # what this step brought to the lender (single tokens are in its stores already)
+            k, v = self.lender.step_kv
         chunk = w.span if (w.span is not None and w.mask_kind == "chunk") else 0
         window = w.span if (w.span is not None and w.mask_kind == "window") else WINDOW_ALL
-        o = ops.seq_swa_attn(q, k, v, kring, vring, pin[:, w.g_off:w.n_in], pin.stride(0), w.scale_h, st, w.H, w.G, w.D,
-                             w.E, window, cap, from_ring_only=single, sink=w.sink, chunk=chunk, softcap=w.softcap,
-                             vfreq=w.v_freq, v_interleaved=w.interleaved)
-        if not single:
+        o = ops.seq_swa_attn(q, k, v, kring, vring, pin[:, w.g_off:w.n_in] if w.gated else None,
+                             pin.stride(0) if w.gated else 0, w.scale_h, st, w.H, w.G, w.D, w.E, window, cap,
+                             from_ring_only=single, sink=w.sink, chunk=chunk, softcap=w.softcap, vfreq=w.v_freq,
+                             v_interleaved=w.interleaved)
+        if own and not single:
             ops.seq_kv_ring_write(k, v, kring, vring, st, cap)
+            self.step_kv = (k, v) if self.lends else None
         return ops.linear(o, w.w_o, out_dtype=F32)
+
+    def end_step(self):
+        """Drops the step's keys and values that other layers may have read."""
+        self.step_kv = None
 
 
 class ValueRotaryAttentionWeights(RotaryAttentionWeights):
@@ -619,6 +679,16 @@ class ValueRotaryAttentionWeights(RotaryAttentionWeights):
 
 class ValueRotaryAttention(RotaryAttention):
     Weights = ValueRotaryAttentionWeights
+
+
+class UnitRotaryAttentionWeights(RotaryAttentionWeights):
+    biases = True
+    gated = False
+    unit_heads = True
+
+
+class UnitRotaryAttention(RotaryAttention):
+    Weights = UnitRotaryAttentionWeights
 
 
 class StateSpaceDualityWeights:
@@ -725,6 +795,8 @@ class ClampedGluFF:
 
 class RoutedExpertsWeights:
     softmax_bias = False  # True: softmax scores, choice on score + `correction`, plain scores as weights
+    top_softmax = False   # True: logits with a bias (`router.b`), choice on the logits, softmax over the chosen ones
+    gated = True          # experts are down(silu(gate x) * (up x)); False: down(relu(up x)^2)
 
     def __init__(self, w, pfx, spec, width, dev, act):
         r = spec["router"]
@@ -745,12 +817,24 @@ class RoutedExpertsWeights:
         if act == torch.bfloat16 and bool((self.router.to(act).to(F32) == self.router).all()):
             pad = (-n_all) % 64
             self.router_act = torch.cat([self.router.to(act), torch.zeros((pad, width), device=dev, dtype=act)]).contiguous()
-        self.w_gate_up = torch.stack([torch.cat([_mat(w, f"{pfx}e{e}.gate", dev, act), _mat(w, f"{pfx}e{e}.up", dev, act)])
-                                      for e in range(self.n)]).contiguous()
+        self.router_bias = None
+        if self.top_softmax:
+            self.router_bias = _vec(w, pfx + "router.b", dev)
+            _expect(pfx, ((self.router_bias, (n_all,)),))
+            if self.router_act is not None:
+                self.router_bias = torch.cat([self.router_bias, torch.zeros(pad, device=dev, dtype=F32)]).contiguous()
+        names = ("gate", "up") if self.gated else ("up",)
+        self.w_up = torch.stack([torch.cat([_mat(w, f"{pfx}e{e}.{n}", dev, act) for n in names])
+                                 for e in range(self.n)]).contiguous()
         self.w_down = torch.stack([_mat(w, f"{pfx}e{e}.down", dev, act) for e in range(self.n)]).contiguous()
         self.correction = _vec(w, pfx + "correction", dev) if self.softmax_bias else None
-        _expect(pfx, ((self.router, (n_all, width)), (self.w_gate_up, (self.n, 2 * ff, width)),
+        _expect(pfx, ((self.router, (n_all, width)), (self.w_up, (self.n, len(names) * ff, width)),
                       (self.w_down, (self.n, width, ff))))
+        self.shared = None
+        if spec.get("shared"):  # one more expert that every token uses, of a size of its own
+            if self.gated:
+                raise ValueError(f"{pfx}: a shared expert is a squared-ReLU unit")
+            self.shared = ReluSquaredFFWeights(w, pfx + "shared.", spec["shared"], width, dev, act)
         if self.correction is not None:
             _expect(pfx, ((self.correction, (n_all,)),))
 
@@ -761,23 +845,38 @@ class RoutedExperts:
 
     def __init__(self, weights, act):
         self.w, self.act = weights, act
+        self.shared = ReluSquaredFF(weights.shared, act) if weights.shared is not None else None
 
     def route(self, x_act):
         w = self.w
         if w.router_act is not None:
-            logits = ops.linear(x_act, w.router_act, out_dtype=F32)[:, :w.n_all]
+            logits = ops.linear(x_act, w.router_act, bias=w.router_bias, out_dtype=F32)[:, :w.n_all]
         else:
-            logits = ops.linear_w32(x_act, w.router)
+            logits = ops.linear_w32(x_act, w.router, bias=w.router_bias)
+        if w.top_softmax:
+            return ops.seq_moe_route_top(logits, w.top)
         return ops.seq_moe_route(logits, w.n_groups, w.keep, w.top, w.scale, softmax_bias=w.softmax_bias,
                                  correction=w.correction)
 
-    def residual(self, x, y, x_act):
-        """x + (y + experts(x_act)): fp32 residual sum with the mixer's output y."""
+    def experts(self, x_act, ids):
+        w = self.w
+        return ops.seq_moe_experts(x_act, ids, w.w_up, w.w_down, n_through=w.n_id, gated=w.gated)
+
+    def terms(self, x_act):
         w = self.w
         if w.n_id:
             raise ValueError("experts that hand their input through need the norm-after-sum residual (post_norm)")
         ids, wts = self.route(x_act)
-        z, pos_of = ops.seq_moe_experts(x_act, ids, w.w_gate_up, w.w_down)
+        z, pos_of = self.experts(x_act, ids)
+        return {"y": self.shared.forward(x_act) if self.shared is not None else None, "z": z, "pos_of": pos_of, "wts": wts}
+
+    def residual(self, x, y, x_act):
+        """x + (y + experts(x_act)): fp32 residual sum with the mixer's output y."""
+        w = self.w
+        if w.n_id or self.shared is not None:
+            raise ValueError("experts that hand their input through, and shared ones, need another residual")
+        ids, wts = self.route(x_act)
+        z, pos_of = self.experts(x_act, ids)
         return ops.seq_residual_combine(x, y, z, pos_of, wts, w.top)
 
     def post_norm(self, x, x_act, alpha, w_norm, eps, act):
@@ -785,8 +884,9 @@ class RoutedExperts:
         inside the norm kernel, in the order of the choices."""
         w = self.w
         ids, wts = self.route(x_act)
-        z, pos_of = ops.seq_moe_experts(x_act, ids, w.w_gate_up, w.w_down, n_through=w.n_id)
-        return ops.seq_post_norm(x, alpha, w_norm, eps, z=z, pos_of=pos_of, wts=wts, ids=ids, n_real=w.n, act=act)
+        z, pos_of = self.experts(x_act, ids)
+        y1 = self.shared.forward(x_act) if self.shared is not None else None
+        return ops.seq_post_norm(x, alpha, w_norm, eps, y1=y1, z=z, pos_of=pos_of, wts=wts, ids=ids, n_real=w.n, act=act)
 
 
 class BiasedSoftmaxExpertsWeights(RoutedExpertsWeights):
@@ -797,10 +897,20 @@ class BiasedSoftmaxExperts(RoutedExperts):
     Weights = BiasedSoftmaxExpertsWeights
 
 
+class TopSoftmaxExpertsWeights(RoutedExpertsWeights):
+    top_softmax = True
+    gated = False
+
+
+class TopSoftmaxExperts(RoutedExperts):
+    Weights = TopSoftmaxExpertsWeights
+
+
 MIXERS = {"attention": GatedWindowAttention, "hgrn2": GatedLinearRecurrence, "latent_attention": LatentWindowAttention,
           "channel_delta": GatedDeltaRule, "general_delta": GeneralizedDeltaRule, "delta": ScalarGatedDeltaRule,
           "sink_attention": SinkAttention, "ssd": StateSpaceDuality, "parallel": ParallelMixers,
           "rotary_attention": RotaryAttention, "rotary_attention_vrot": ValueRotaryAttention,
+          "rotary_attention_unit": UnitRotaryAttention,
           "latent_attention_causal": LatentCausalAttention}
 FEED_FORWARDS = {"dense": ReluSquaredFF, "moe": RoutedExperts, "clamped_glu": ClampedGluFF,
-                 "moe_softmax_bias": BiasedSoftmaxExperts}
+                 "moe_softmax_bias": BiasedSoftmaxExperts, "relu_glu": ReluGluFF, "moe_top_softmax": TopSoftmaxExperts}

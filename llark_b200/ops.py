@@ -9,7 +9,8 @@ import math
 
 import torch
 
-from ._lib import EPI_QUICK_GELU, EPI_ROPE, EPI_SWIGLU_BWD, GemmEpilogue, check, lib
+from ._lib import (EPI_NONE, EPI_QUICK_GELU, EPI_RELU2, EPI_RELU_GLU, EPI_ROPE, EPI_SWIGLU_BWD, GemmEpilogue, check,
+                   lib)
 
 BF16 = torch.bfloat16
 
@@ -48,12 +49,13 @@ def _req(t, dtype=None):
 
 def gemm(a, b, *, a_mn=False, b_mn=False, M=None, N=None, K=None, out=None, out_dtype=None, bias=None,
          residual=None, lda=None, ldb=None, ldc=None, ldr=None, max_ctas=0, quick_gelu=False, rope=None,
-         swiglu_bwd=None):
+         swiglu_bwd=None, act=None):
     """C[M,N] = A[M,K] @ B[N,K]^T (+bias) (+residual), optionally with one fused epilogue (llark_gemm_ex):
 
     quick_gelu=True            C = quick_gelu(acc + bias)
     rope=(cos, sin, S, cols)   columns [0, cols) rotated per 128-wide head, position = row % S (fused-QKV projection)
     swiglu_bwd=gu              acc is d(act) [M, I]; `out` must be the dgu buffer [M, 2I]: out = (dgate | dup)
+    act="relu2" | "relu_glu"   see linear()
 
     a: [M,K] (a_mn=False) or [K,M] (a_mn=True); b: [N,K] (b_mn=False) or [K,N] (b_mn=True); row-major with
     leading dimension = last-dim stride unless lda/ldb given. bf16 inputs use kind::f16, fp32 inputs kind::tf32.
@@ -96,6 +98,8 @@ def gemm(a, b, *, a_mn=False, b_mn=False, M=None, N=None, K=None, out=None, out_
         ep = GemmEpilogue(EPI_ROPE, cos_t.data_ptr(), sin_t.data_ptr(), 0, int(S_rope), int(cols))
     elif swiglu_bwd is not None:
         ep = GemmEpilogue(EPI_SWIGLU_BWD, swiglu_bwd.data_ptr(), None, swiglu_bwd.stride(0), 0, 0)
+    elif act is not None:
+        ep = GemmEpilogue({"relu2": EPI_RELU2, "relu_glu": EPI_RELU_GLU}[act], None, None, 0, 0, 0)
     if ep is None:
         rc = lib().llark_gemm(_p(a), int(a_mn), lda, _p(b), int(b_mn), ldb, _p(out), ldc, int(c_fp32), _p(bias),
                               int(bias_fp32), _p(residual), ldr, M, N, K, int(in_fp32), max_ctas, _stream())
@@ -483,9 +487,13 @@ LINEAR_ROWS_MAX = 8
 LINEAR_STATS = {"rows": 0, "tcgen05": 0, "simt": 0}
 
 
-def linear(a, w, bias=None, out_dtype=None, out=None):
-    """y[M, N] = a[M, K] @ w[N, K]^T (+ bias fp32 [N]); a and w both bf16 or both fp32 (true fp32 arithmetic, no TF32);
-    output bf16 or fp32."""
+LINEAR_ACTS = {None: 0, "relu2": 1, "relu_glu": 2}
+
+
+def linear(a, w, bias=None, out_dtype=None, out=None, act=None):
+    """y[M, N] = act(a[M, K] @ w[N, K]^T (+ bias fp32 [N])); a and w both bf16 or both fp32 (true fp32 arithmetic, no TF32);
+    output bf16 or fp32. act, applied to the fp32 sums before the one rounding: "relu2" = relu(z)^2; "relu_glu": the rows of
+    w alternate gate, up and y [M, N / 2] = relu(z[:, 2c]) * z[:, 2c + 1]."""
     _req(a), _req(w)
     if a.dtype != w.dtype:
         raise TypeError("linear: activation and weight dtypes differ")
@@ -494,8 +502,11 @@ def linear(a, w, bias=None, out_dtype=None, out=None):
     N = w.shape[0]
     if w.shape[1] != K:
         raise ValueError("linear: inner sizes differ")
+    code = LINEAR_ACTS[act]
+    if act == "relu_glu" and N % 2:
+        raise ValueError("linear: gate and up rows must come in pairs")
     if out is None:
-        out = torch.empty((M, N), device=a.device, dtype=out_dtype or a.dtype)
+        out = torch.empty((M, N // 2 if act == "relu_glu" else N), device=a.device, dtype=out_dtype or a.dtype)
     c_fp32 = _actf(out.dtype)
     if bias is not None:
         _req(bias, torch.float32)
@@ -503,15 +514,15 @@ def linear(a, w, bias=None, out_dtype=None, out=None):
     if M <= LINEAR_ROWS_MAX:
         LINEAR_STATS["rows"] += 1
         check(lib().llark_linear_rows(_p(a), a.stride(0), _p(w), w.stride(0), _p(out), out.stride(0), c_fp32, _p(bias),
-                                      M, N, K, in_fp32, _stream()), "linear_rows")
-    elif (not in_fp32 and K >= 64 and N >= 64 and K % 8 == 0 and a.stride(0) % 8 == 0 and w.stride(0) % 8 == 0 and out.stride(0) % vec == 0
+                                      M, N, K, in_fp32, code, _stream()), "linear_rows")
+    elif (not in_fp32 and not (c_fp32 and act == "relu_glu") and K >= 64 and N >= 64 and K % 8 == 0 and a.stride(0) % 8 == 0 and w.stride(0) % 8 == 0 and out.stride(0) % vec == 0
           and a.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0 and out.data_ptr() % 16 == 0):
         LINEAR_STATS["tcgen05"] += 1
-        gemm(a, w, bias=bias, out=out, M=M, N=N, K=K)
+        gemm(a, w, bias=bias, out=out, M=M, N=N, K=K, act=act)
     else:
         LINEAR_STATS["simt"] += 1
         check(lib().llark_linear_simt(_p(a), a.stride(0), _p(w), w.stride(0), _p(out), out.stride(0), c_fp32, _p(bias),
-                                      M, N, K, in_fp32, _stream()), "linear_simt")
+                                      M, N, K, in_fp32, code, _stream()), "linear_simt")
     return out
 
 
@@ -567,6 +578,37 @@ def seq_gated_norm_add(x, y, w, eps, gate=None, w_next=None, act=None):
                                          _p(w_next), _p(out), _p(xa), rows, C, float(eps),
                                          _actf(act) if w_next is not None else 0, _stream()), "seq_gated_norm_add")
     return (out, xa) if w_next is not None else out
+
+
+def seq_tanh_norm(x, norm, act, rows=None):
+    """tanh(alpha * x) * w + b of fp32 rows in `act`, norm = (alpha, w fp32 [C], b fp32 [C]); rows: int32 row numbers (all
+    when None)."""
+    alpha, w, b = norm
+    _req(x, torch.float32), _req(w, torch.float32), _req(b, torch.float32)
+    n, C = (rows.numel() if rows is not None else x.shape[0]), x.shape[1]
+    out = torch.empty((n, C), device=x.device, dtype=act)
+    check(lib().llark_seq_tanh_norm(_p(x), _p(rows), float(alpha), _p(w), _p(b), _p(out), n, C, _actf(act), _stream()),
+          "seq_tanh_norm")
+    return out
+
+
+def seq_tanh_norm_add(x, post, y=None, z=None, pos_of=None, wts=None, next_norm=None, act=None):
+    """x + tanh(alpha * f) * w + b (fp32, new tensor), post = (alpha, w, b), f = y + the weighted sum of the chosen experts'
+    outputs (z, pos_of, wts [n_tok, top]; either part may be missing); with next_norm = (alpha, w, b) also the next
+    sublayer's input, the tanh norm of the result in `act`."""
+    _req(x, torch.float32)
+    rows, C = x.shape
+    for t in (y, z):
+        if t is not None and (not _req(t, torch.float32).is_contiguous() or t.shape[1] != C):
+            raise ValueError("seq_tanh_norm_add: sublayer results must be contiguous and of the stream's width")
+    out = torch.empty_like(x)
+    xa = torch.empty((rows, C), device=x.device, dtype=act) if next_norm is not None else None
+    alpha, w, b = post
+    na, nw, nb = next_norm if next_norm is not None else (0.0, None, None)
+    check(lib().llark_seq_tanh_norm_add(_p(x), _p(y), _p(z), _p(pos_of), _p(wts), wts.shape[1] if wts is not None else 0,
+                                        float(alpha), _p(w), _p(b), float(na), _p(nw), _p(nb), _p(out), _p(xa), rows, C,
+                                        _actf(act) if next_norm is not None else 0, _stream()), "seq_tanh_norm_add")
+    return (out, xa) if next_norm is not None else out
 
 
 def seq_rmsnorm_rows(x, rows, w, eps, act):
@@ -651,24 +693,25 @@ def seq_swa_attn(qn, kn, vv, kring, vring, gate, gate_ld, scale_h, st, H, G, D, 
 
 
 def seq_qkv_rotary(src, q_off, k_off, v_off, H, G, D, E, eps, act, st, wq=None, wk=None, qk_freq=None, qk_interleaved=False,
-                   v_freq=None, v_interleaved=False, kring=None, vring=None, cap=0):
+                   v_freq=None, v_interleaved=False, kring=None, vring=None, cap=0, unit=False):
     """src fp32 [n_tok, ld] -> (q [n_tok, H*D], k [n_tok, G*D], v [n_tok, G*E]) in `act`. wq / wk: RMS norm over the whole
     q / k projection with weights [H*D] / [G*D]. qk_freq fp32 [n_rot / 2]: the first n_rot entries of each q / k head are
     rotated by position * frequency (pairs (i, i + n_rot/2), or (2i, 2i+1) when interleaved). v_freq fp32 [E / 2]: the
-    value heads are rotated the same way over all of E. With kring / vring the k / v rows also go straight into the rings
-    (steps of one token per request)."""
+    value heads are rotated the same way over all of E. unit: every rotated q / k head is divided by its root mean square.
+    G = 0: queries only (k = v = None). With kring / vring the k / v rows also go straight into the rings (steps of one
+    token per request)."""
     _req(src, torch.float32)
     n = src.shape[0]
     qn = torch.empty((n, H * D), device=src.device, dtype=act)
-    kn = torch.empty((n, G * D), device=src.device, dtype=act)
-    vv = torch.empty((n, G * E), device=src.device, dtype=act)
+    kn = torch.empty((n, G * D), device=src.device, dtype=act) if G else None
+    vv = torch.empty((n, G * E), device=src.device, dtype=act) if G else None
     n_rot = 2 * qk_freq.numel() if qk_freq is not None else 0
     if v_freq is not None and v_freq.numel() != E // 2:
         raise ValueError("seq_qkv_rotary: one frequency per pair of value channels")
     check(lib().llark_seq_qkv_rotary(_p(src), src.stride(0), q_off, k_off, v_off, _p(wq), _p(wk), _p(qk_freq), n_rot,
                                      int(qk_interleaved), _p(v_freq), int(v_interleaved), _p(qn), _p(kn), _p(vv), _p(kring),
                                      _p(vring), _p(st.tok_seq), _p(st.cu), _p(st.pos0), _p(st.slot), n, H, G, D, E, int(cap),
-                                     float(eps), _actf(act), _stream()), "seq_qkv_rotary")
+                                     float(eps), int(unit), _actf(act), _stream()), "seq_qkv_rotary")
     return qn, kn, vv
 
 
@@ -898,20 +941,30 @@ def seq_moe_route(logits, n_groups, keep, top, scale, softmax_bias=False, correc
     return ids, wts
 
 
+def seq_moe_route_top(logits, top):
+    """The `top` largest logits of each row: expert numbers int32 [n, top] and weights fp32 [n, top] = softmax over them."""
+    n, n_exp = logits.shape
+    ids = torch.empty((n, top), device=logits.device, dtype=torch.int32)
+    wts = torch.empty((n, top), device=logits.device, dtype=torch.float32)
+    check(lib().llark_seq_moe_route_top(_p(_req(logits, torch.float32)), logits.stride(0), _p(ids), _p(wts), n, n_exp,
+                                        int(top), _stream()), "seq_moe_route_top")
+    return ids, wts
+
+
 # entries (tokens x choices) from which a bf16 step runs every expert's rows through the tcgen05 GEMM core; smaller steps,
 # and fp32, stay on the grouped SIMT kernels. Neither route reads anything back to the host.
 MOE_DENSE_MIN_ENTRIES = 2048
 
 
-def seq_moe_experts(x, ids, w_gate_up, w_down, n_through=0):
-    """x act [n_tok, C]; ids int32 [n_tok, top]; w_gate_up act [n_exp, 2*ff, C] (gate rows, then up rows);
-    w_down act [n_exp, C, ff] -> (z fp32 [n_tok*top, C] expert outputs in sorted order, pos_of int32 [n_tok*top]).
+def seq_moe_experts(x, ids, w_up, w_down, n_through=0, gated=True):
+    """x act [n_tok, C]; ids int32 [n_tok, top]; w_up act [n_exp, 2*ff, C] (gate rows, then up rows; silu(gate x) * (up x))
+    or, not gated, [n_exp, ff, C] (relu(up x)^2); w_down act [n_exp, C, ff] -> (z fp32 [n_tok*top, C] expert outputs in sorted order, pos_of int32 [n_tok*top]).
     n_through: expert numbers n_exp .. n_exp + n_through - 1 have no weights; their rows of z are not written."""
     L = lib()
     n_tok, top = ids.shape
-    n_real, ff2, C = w_gate_up.shape
+    n_real, n_up, C = w_up.shape
     n_exp = n_real + int(n_through)
-    ff = ff2 // 2
+    ff = n_up // 2 if gated else n_up
     n_ent = n_tok * top
     dense = (x.dtype == BF16 and n_ent >= MOE_DENSE_MIN_ENTRIES and C % 8 == 0 and ff % 8 == 0 and C >= 64 and ff >= 64
              and L.llark_gemm_get_mode() == 1)
@@ -937,15 +990,16 @@ def seq_moe_experts(x, ids, w_gate_up, w_down, n_through=0):
         count = meta[1:]
         xs = torch.empty((n_ent, C), device=x.device, dtype=x.dtype)
         check(L.llark_seq_moe_gather(_p(x), x.stride(0), _p(perm), top, _p(xs), n_ent, C, 0, _stream()), "seq_moe_gather")
-        gu = torch.empty((n_ent, ff2), device=x.device, dtype=x.dtype)
-        check(L.llark_gemm_segments(_p(xs), C, _p(w_gate_up), _p(gu), ff2, 0, None, n_real, _p(tiles256), max256, _p(count),
-                                    n_ent, ff2, C, _stream()), "gemm_segments(gate|up)")
-        check(L.llark_seq_silu_mul(_p(gu), _p(act), n_ent, ff, 0, _stream()), "seq_silu_mul")
+        gu = torch.empty((n_ent, n_up), device=x.device, dtype=x.dtype) if gated else act
+        check(L.llark_gemm_segments(_p(xs), C, _p(w_up), _p(gu), n_up, 0, None, n_real, _p(tiles256), max256, _p(count),
+                                    n_ent, n_up, C, EPI_NONE if gated else EPI_RELU2, _stream()), "gemm_segments(up)")
+        if gated:
+            check(L.llark_seq_silu_mul(_p(gu), _p(act), n_ent, ff, 0, _stream()), "seq_silu_mul")
         check(L.llark_gemm_segments(_p(act), ff, _p(w_down), _p(z), C, 1, None, n_real, _p(tiles256), max256, _p(count),
-                                    n_ent, C, ff, _stream()), "gemm_segments(down)")
+                                    n_ent, C, ff, EPI_NONE, _stream()), "gemm_segments(down)")
         return z, pos_of
-    check(L.llark_seq_moe_up(_p(x), x.stride(0), _p(perm), top, _p(w_gate_up), _p(act), _p(tiles), _p(meta), max_tiles,
-                             n_ent, ff, C, _actf(x.dtype), _stream()), "seq_moe_up")
+    check(L.llark_seq_moe_up(_p(x), x.stride(0), _p(perm), top, _p(w_up), _p(act), _p(tiles), _p(meta), max_tiles,
+                             n_ent, ff, C, int(gated), _actf(x.dtype), _stream()), "seq_moe_up")
     check(L.llark_seq_moe_down(_p(act), _p(w_down), _p(z), _p(tiles), _p(meta), max_tiles, n_ent, C, ff, _actf(x.dtype),
                                _stream()), "seq_moe_down")
     return z, pos_of

@@ -1,6 +1,7 @@
 """Generation throughput of the Kelutar path beside the Llama path at equal size (`bench.py --workload generation`), of
-Golavik beside Kelutar (`generation-golavik`), of Gubulorn beside Golavik (`generation-gubulorn`) and of Tokatar beside an
-all-attention Kelutar (`generation-tokatar`).
+Golavik beside Kelutar (`generation-golavik`), of Gubulorn beside Golavik (`generation-gubulorn`), of Tokatar beside an
+all-attention Kelutar (`generation-tokatar`) and of Manapel beside an all-attention Tokatar and a Golavik with the same
+experts (`generation-manapel`).
 
 Random weights, synthetic token ids. For each size: prefill tokens/s (a packed batch of whole prompts) and decode tokens/s
 (one token per request and step, after a prompt of `context` tokens) for both decoders, plus a per-op table: every op
@@ -191,11 +192,11 @@ def _op_work(name, a, k, out, ctx):
         per = 9.0 if k.get("correct", True) else 5.0  # without the correction: decay, write and read-out only
         return (_nbytes(vec) + st.n_tok * H * E * 8 + 2 * st.n_seq * H * D * E * 4), per * st.n_tok * H * D * E
     if name == "seq_moe_experts":
-        x, ids, wgu, wd = a[0], a[1], a[2], a[3]
-        n_ent, (n_exp, ff2, C) = ids.numel(), wgu.shape
+        x, ids, wup, wd = a[0], a[1], a[2], a[3]
+        n_ent, (n_exp, n_up, C), ff = ids.numel(), wup.shape, wd.shape[2]
         hit = min(n_exp, n_ent)
-        return (hit * (ff2 * C + C * ff2 // 2) * wgu.element_size() + n_ent * C * (x.element_size() + 4)
-                + n_ent * ff2 * x.element_size()), 2.0 * n_ent * 3 * (ff2 // 2) * C
+        return (hit * (n_up + ff) * C * wup.element_size() + n_ent * C * (x.element_size() + 4)
+                + 2 * n_ent * ff * x.element_size()), 2.0 * n_ent * (n_up + ff) * C
     if name == "seq_head_linear":
         x, w, y, N, K = a[0], a[2], a[3], k["N"], k["K"]
         M, H = x.shape[0], w.shape[0]
@@ -219,6 +220,8 @@ def _op_work(name, a, k, out, ctx):
 
 
 def op_table(records, ctx, peaks):
+    from llark_b200 import ops
+
     bw, fl = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
     agg = {}
     for name, e0, e1, a, k, out in records:
@@ -227,7 +230,8 @@ def op_table(records, ctx, peaks):
         ms = e0.elapsed_time(e1)
         nb, flops = _op_work(name, a, k, out, ctx)
         if name == "linear":
-            name = "linear_rows" if a[0].shape[0] <= 8 else "linear_tcgen05"
+            M, K = a[0].shape
+            name = "linear_rows" if M <= 8 and ops.linear_rows_pays(M, a[1].shape[0], K) else "linear_tcgen05"
         if name == "gemm":
             name = "gemm_tcgen05"
         d = agg.setdefault(name, {"calls": 0, "ms": 0.0, "bytes": 0, "flops": 0.0, "roof_ms": 0.0})
@@ -642,6 +646,117 @@ def run_tokatar(args, peaks, peaks_kind, emit):
           "warmup": max(args.warmup, 3), "ms_per_step": head["prefill"]["tokatar_ms"], "higher_is_better": True,
           "scaling": "weak", "vs_baseline": None, "dtype": "bf16", "data": "synthetic token ids, random weights",
           "config": {"model": "Tokatar " + head["size"], "l2": "256 MB fill between timed steps",
+                     "peaks": peaks_kind, "hbm_gbs": peaks["hbm_gbs"], "bf16_tflops": peaks["bf16_tflops"]},
+          "sizes": results, "wall_s": round(time.time() - t0, 1)})
+
+
+MANAPEL_OPS = ["linear", "linear_w32", "seq_embed", "seq_tanh_norm", "seq_tanh_norm_add", "seq_qkv_rotary", "seq_swa_attn",
+               "seq_kv_ring_write", "seq_moe_route_top", "seq_moe_experts"]
+
+# (name, width, layers, heads, key/value heads, head dim, dense ff, experts, top, expert ff, shared ff, vocab): the first layer
+# has the dense feed-forward, the others experts; every second layer reads the keys and values of the one before it. Beside
+# it: a Tokatar model with attention over everything before in every layer (same width, layers, heads, key / value heads; a
+# feed-forward of top x expert ff + shared ff rows), and a Golavik model with the same width, layers, heads and experts.
+MANAPEL_SIZES = [
+    ("m2048", 2048, 4, 16, 4, 128, 8192, 32, 4, 1024, 2048, 32000),
+    ("m4096", 4096, 4, 32, 8, 128, 11008, 64, 6, 1024, 2048, 32000),
+]
+
+
+def manapel_config(width, layers, heads, kv, dim, dense, experts, top, ff, shared, vocab):
+    ls = []
+    for i in range(layers):
+        m = {"heads": heads, "kv_heads": kv, "dim": dim, "vdim": dim, "scale": 1.0 / math.sqrt(dim),
+             "rot": {"base": 100000.0, "dims": dim}}
+        if i % 2:
+            m["kv_from"] = i - 1
+        mlp = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top}, "shared": {"ff": shared}}
+        ls.append({"type": "attention", "mixer": m, "mlp": mlp if i else {"kind": "dense", "ff": dense}})
+    return {"architecture": "Manapel", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "logit_scale": 1.0, "layers": ls}
+
+
+def manapel_random_weights(cfg, device, seed=0):
+    g = torch.Generator(device=device).manual_seed(seed)
+    C = cfg["width"]
+
+    def mat(o, i, s=None):
+        return (torch.randn(o, i, device=device, generator=g) * (s or 1.0 / math.sqrt(i))).to(BF16)
+
+    def vec(n, mean=1.0, s=0.1):
+        return (mean + torch.randn(n, device=device, generator=g) * s).to(BF16)
+
+    W = {"embed": mat(cfg["vocab"], C, 1.0), "head": mat(cfg["vocab"], C)}
+    names = ["final.norm"]
+    for i, layer in enumerate(cfg["layers"]):
+        p, m, mlp = "l%d." % i, layer["mixer"], layer["mlp"]
+        names += [p + n for n in ("norm1", "norm1b", "norm2", "norm2b")]
+        rows = {"q": m["heads"] * m["dim"]}
+        if "kv_from" not in m:
+            rows.update(k=m["kv_heads"] * m["dim"], v=m["kv_heads"] * m["vdim"])
+        for n, r in rows.items():
+            W.update({p + "mix." + n: mat(r, C), p + "mix." + n + ".b": vec(r, 0.0)})
+        W[p + "mix.o"] = mat(C, m["heads"] * m["vdim"])
+        if mlp["kind"] == "dense":
+            units = {"": mlp["ff"]}
+            W[p + "mlp.gate"] = mat(mlp["ff"], C)
+        else:
+            n = mlp["router"]["experts"]
+            units = {"e%d." % e: mlp["expert"]["ff"] for e in range(n)}
+            units["shared."] = mlp["shared"]["ff"]
+            W.update({p + "mlp.router": mat(n, C), p + "mlp.router.b": vec(n, 0.0)})
+        for u, f in units.items():
+            W.update({p + "mlp." + u + "up": mat(f, C), p + "mlp." + u + "down": mat(C, f)})
+    for n in names:
+        W.update({n: vec(C), n + ".b": vec(C, 0.0), n + ".alpha": vec(1, 0.5).reshape(())})
+    return W
+
+
+def bench_size_manapel(name, width, layers, heads, kv, dim, dense, experts, top, ff, shared, vocab, peaks, steps, warmup,
+                       prefill_batch=4, prompt=2048, decode_batches=(1, 8, 32), context=1024):
+    """Manapel beside the two existing decoders that share its parts: an all-attention Tokatar (norms around each sublayer,
+    rotary attention over everything before, dense feed-forward) and a Golavik (routed experts)."""
+    from llark_b200.models.golavik import GolavikConfig, GolavikForCausalLM
+    from llark_b200.models.manapel import ManapelConfig, ManapelForCausalLM
+    from llark_b200.models.tokatar import TokatarConfig, TokatarForCausalLM
+
+    flush = _Flush()
+    out = {"size": name, "width": width, "layers": layers, "heads": heads, "kv_heads": kv, "head_dim": dim, "dense_ff": dense,
+           "experts": experts, "top": top, "expert_ff": ff, "shared_ff": shared, "vocab": vocab,
+           "prefill": {"batch": prefill_batch, "prompt": prompt}, "decode": {"context": context}}
+    g = torch.Generator().manual_seed(0)
+    tcfg = tokatar_config(width, layers, heads, kv, dim, None, top * ff + shared, 192, 64, vocab)
+    att = tcfg["layers"][0]
+    del att["mixer"]["mask"], att["mixer"]["softcap"]
+    tcfg["layers"] = [att] * layers
+    mcfg = manapel_config(width, layers, heads, kv, dim, dense, experts, top, ff, shared, vocab)
+    gcfg = golavik_config(width, layers, heads, dim, max(prompt, context), experts, top, ff, 192, 64, vocab)
+    for tag, cls, conf, cfg, weights, op_names in (
+            ("manapel", ManapelForCausalLM, ManapelConfig, mcfg, manapel_random_weights, MANAPEL_OPS),
+            ("tokatar", TokatarForCausalLM, TokatarConfig, tcfg, tokatar_random_weights, TOKATAR_OPS),
+            ("golavik", GolavikForCausalLM, GolavikConfig, gcfg, golavik_random_weights, GOLAVIK_OPS)):
+        m = cls(conf.from_dict(cfg), weights(cfg, "cuda"), dtype=BF16)
+        m.engine.max_positions = max(prompt, context) + 64
+        bench_native(tag, m.engine, op_names, out, vocab, peaks, steps, warmup, flush, g, prefill_batch, prompt,
+                     decode_batches, context)
+        del m
+        torch.cuda.empty_cache()
+    return out
+
+
+def run_manapel(args, peaks, peaks_kind, emit):
+    from llark_b200 import ops
+
+    ops.init()
+    t0 = time.time()
+    sizes = [s for s in MANAPEL_SIZES if not os.environ.get("LLARK_BENCH_SIZE") or s[0] == os.environ["LLARK_BENCH_SIZE"]]
+    results = [bench_size_manapel(*s, peaks=peaks, steps=args.steps, warmup=max(args.warmup, 3)) for s in sizes]
+    head = results[0]
+    emit({"metric": "generation tokens/s, Manapel beside an all-attention Tokatar at equal size (prefill of %d x %d tokens)"
+                    % (head["prefill"]["batch"], head["prefill"]["prompt"]),
+          "value": head["prefill"]["manapel_tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "steps": args.steps,
+          "warmup": max(args.warmup, 3), "ms_per_step": head["prefill"]["manapel_ms"], "higher_is_better": True,
+          "scaling": "weak", "vs_baseline": None, "dtype": "bf16", "data": "synthetic token ids, random weights",
+          "config": {"model": "Manapel " + head["size"], "l2": "256 MB fill between timed steps",
                      "peaks": peaks_kind, "hbm_gbs": peaks["hbm_gbs"], "bf16_tflops": peaks["bf16_tflops"]},
           "sizes": results, "wall_s": round(time.time() - t0, 1)})
 

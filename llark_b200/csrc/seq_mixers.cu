@@ -385,6 +385,115 @@ __global__ void qkv_rotary4_kernel(const float* __restrict__ src, long long ld, 
     }
 }
 
+// The same for unit heads with pairs in halves and plain values, one read of every entry: a group of GS lanes owns a head of
+// one token, NI work items per lane (item j: quads j and j + n_rot / 8 of the rotated zone, then the quads behind it), which
+// wait in registers while the group adds up its squares; a token's values are copied in runs of 2 GS NI quads, whatever their
+// heads. A block takes `tb` tokens: it builds their tables of angles at once, and then its groups walk the tokens' heads and
+// runs without another barrier.
+template <typename T, int GS, int NI>
+__global__ void __launch_bounds__(512)
+qkv_unit4_kernel(const float* __restrict__ src, long long ld, int q_off, int k_off, int v_off,
+                 const float* __restrict__ qk_freq, int n_rot, T* __restrict__ qn, T* __restrict__ kn, T* __restrict__ vv,
+                 T* __restrict__ kring, T* __restrict__ vring, const int* __restrict__ tok_seq,
+                 const int* __restrict__ cu, const int* __restrict__ pos0, const int* __restrict__ slot, int n_tok, int tb,
+                 int H, int G, int D, int E, int cap, float eps) {
+    extern __shared__ float cs[];  // [tb][n_rot]: cos, sin per pair
+    const int t0 = blockIdx.x * tb, nt = n_tok - t0 < tb ? n_tok - t0 : tb;
+    constexpr int RUN = 2 * GS * NI;
+    const int nq = n_rot >> 3, iq = nq + ((D - n_rot) >> 2), vq = (G * E) >> 2, half = n_rot >> 1;
+    const int sub = threadIdx.x / GS, l = threadIdx.x % GS, ns = blockDim.x / GS;
+    const int heads = H + G + (vq + RUN - 1) / RUN, total = nt * heads;
+    auto position = [&](int t) {
+        const int b = tok_seq[t];
+        return (long long)pos0[b] + (t - cu[b]);
+    };
+    float4 a[NI], c[NI];
+    auto load = [&](int w) {
+        const int tok = w / heads, hh = w - tok * heads;
+        const bool val = hh >= H + G;
+        const float4* s = reinterpret_cast<const float4*>(
+            src + (long long)(t0 + tok) * ld +
+            (hh < H ? q_off + hh * D : (val ? v_off : k_off + (hh - H) * D)));
+        const int v0 = (hh - H - G) * RUN + l;
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+            const int j = l + i * GS;
+            a[i] = c[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (w >= total) continue;
+            if (val) {
+                if (v0 + 2 * i * GS < vq) a[i] = s[v0 + 2 * i * GS];
+                if (v0 + (2 * i + 1) * GS < vq) c[i] = s[v0 + (2 * i + 1) * GS];
+            } else if (j < nq) {
+                a[i] = s[j];
+                c[i] = s[nq + j];
+            } else if (j < iq) {
+                a[i] = s[nq + j];  // 2 * nq + (j - nq)
+            }
+        }
+    };
+    load(sub);
+    for (int i = threadIdx.x; i < nt * half; i += blockDim.x) {
+        const int tok = i / half, k = i - tok * half;
+        sincosf((float)position(t0 + tok) * qk_freq[k], &cs[2 * i + 1], &cs[2 * i]);
+    }
+    __syncthreads();
+    for (int base = 0; base < total; base += ns) {  // the same number of passes for every lane of a warp
+        const int w = base + sub;
+        if (base) load(w);
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+            ss += a[i].x * a[i].x + a[i].y * a[i].y + a[i].z * a[i].z + a[i].w * a[i].w;
+            ss += c[i].x * c[i].x + c[i].y * c[i].y + c[i].z * c[i].z + c[i].w * c[i].w;
+        }
+#pragma unroll
+        for (int m = GS / 2; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
+        if (w >= total) continue;
+        const int tok = w / heads, hh = w - tok * heads;
+        const long long t = t0 + tok;
+        const bool val = hh >= H + G;
+        const float r = val ? 1.f : 1.0f / sqrtf(ss / (float)D + eps);
+        T *o, *o2 = nullptr;
+        if (hh < H) {
+            o = qn + (t * H + hh) * D;
+        } else {
+            o = val ? vv + t * G * E : kn + (t * G + hh - H) * D;
+            if (kring) {
+                const long long e = (long long)slot[tok_seq[t]] * cap + (position((int)t) % cap);
+                o2 = val ? vring + e * G * E : kring + (e * G + hh - H) * D;
+            }
+        }
+        auto put = [&](int quad, const float (&v)[4]) {
+            st_quad(o + 4 * quad, v);
+            if (o2) st_quad(o2 + 4 * quad, v);
+        };
+        const float2* angles = reinterpret_cast<const float2*>(cs) + tok * half;
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+            const int j = l + i * GS;
+            const float u[4] = {a[i].x * r, a[i].y * r, a[i].z * r, a[i].w * r};
+            const float v[4] = {c[i].x * r, c[i].y * r, c[i].z * r, c[i].w * r};
+            if (val) {
+                const int q0 = (hh - H - G) * RUN + l + 2 * i * GS;
+                if (q0 < vq) put(q0, u);
+                if (q0 + GS < vq) put(q0 + GS, v);
+            } else if (j < nq) {
+                float x[4], y[4];
+#pragma unroll
+                for (int k = 0; k < 4; ++k) {
+                    const float2 an = angles[4 * j + k];
+                    x[k] = u[k] * an.x - v[k] * an.y;
+                    y[k] = v[k] * an.x + u[k] * an.y;
+                }
+                put(j, x);
+                put(nq + j, y);
+            } else if (j < iq) {
+                put(nq + j, u);
+            }
+        }
+    }
+}
+
 // N consecutive elements -> float, with one 4 / 8 / 16-byte load per piece when `vec` (the address is then aligned to
 // the piece); scalar loads otherwise.
 template <typename T, int N>
@@ -878,6 +987,34 @@ extern "C" int llark_seq_qkv_rotary(const float* src, long long ld, int q_off, i
     if (quads) items /= 4;
     int threads = n_tok >= 1024 ? 256 : (items + 31) / 32 * 32;
     threads = threads < 64 ? 64 : (threads > 1024 ? 1024 : threads);
+    const int per = n_rot / 8 + (D - n_rot) / 4;  // work items of a rotated head
+    if (unit && quads && !qk_interleaved && !v_freq && per <= 64) {
+        const int gs = per <= 8 ? 8 : (per <= 16 ? 16 : 32);
+        // many tokens: four per block, whose groups of lanes walk the heads; few (decoding): a group for every head
+        int tb = n_tok >= 1024 ? 4 : 1;
+        while (tb > 1 && sizeof(float) * (size_t)tb * n_rot > 16 * 1024) tb >>= 1;
+        int th = ((H + 2 * G) * gs + 31) / 32 * 32;
+        th = tb > 1 ? 256 : (th > 512 ? 512 : th);
+        const unsigned blocks = (unsigned)((n_tok + tb - 1) / tb);
+        const size_t table = sizeof(float) * (size_t)tb * n_rot;
+#define LLARK_UNIT(T, GS, NI)                                                                                         \
+    qkv_unit4_kernel<T, GS, NI><<<blocks, th, table, st>>>(src, ld, q_off, k_off, v_off, qk_freq, n_rot, (T*)qn, (T*)kn, \
+                                                           (T*)vv, (T*)kring, (T*)vring, tok_seq, cu, pos0, slot, n_tok, \
+                                                           tb, H, G, D, E, cap, eps)
+        if (act_fp32) {
+            if (per <= 8) LLARK_UNIT(float, 8, 1);
+            else if (per <= 16) LLARK_UNIT(float, 16, 1);
+            else if (per <= 32) LLARK_UNIT(float, 32, 1);
+            else LLARK_UNIT(float, 32, 2);
+        } else {
+            if (per <= 8) LLARK_UNIT(bf16_t, 8, 1);
+            else if (per <= 16) LLARK_UNIT(bf16_t, 16, 1);
+            else if (per <= 32) LLARK_UNIT(bf16_t, 32, 1);
+            else LLARK_UNIT(bf16_t, 32, 2);
+        }
+#undef LLARK_UNIT
+        return check_launch();
+    }
 #define LLARK_ROTARY(KERNEL, T)                                                                                      \
     KERNEL<T><<<n_tok, threads, smem, st>>>(src, ld, q_off, k_off, v_off, wq, wk, qk_freq, n_rot, qk_interleaved, v_freq, \
                                             v_interleaved, (T*)qn, (T*)kn, (T*)vv, (T*)kring, (T*)vring, tok_seq, cu, pos0, \

@@ -377,22 +377,24 @@ grouped_linear_kernel(const T* __restrict__ A, long long lda, const int* __restr
         }
 }
 
-// Few rows per expert (decode): a warp owns one output column of one row tile and streams its weight row (kSiluGlu: the gate
-// and the up row) once in 16-byte pieces; the tile's rows come from L1 / L2, eight at a time.
-template <typename T, typename TC, int MODE>
+// Few rows per expert (decode): a warp owns one output column of one row tile (kSiluGlu: its gate and its up row) or two
+// adjacent ones (kPlain, kRelu2) and streams the two weight rows in 16-byte pieces; the tile's rows come from L1 / L2, MB at a
+// time, and are read once for both. A small MB keeps the registers few and the warps many, which pays as long as an expert
+// has a handful of rows (the second pass over a weight row comes from L1).
+template <typename T, typename TC, int MODE, int MB>
 __global__ void __launch_bounds__(256)
 grouped_rows_kernel(const T* __restrict__ A, long long lda, const int* __restrict__ perm, int top,
                     const T* __restrict__ W, TC* __restrict__ Cm, long long ldc, const int* __restrict__ tiles,
                     const int* __restrict__ meta, int N, int K, int vec_ok) {
-    constexpr int MB = 8, VEC = 16 / (int)sizeof(T);
+    constexpr int VEC = 16 / (int)sizeof(T);
     constexpr bool DUAL = MODE == kSiluGlu;
     if ((int)blockIdx.y >= meta[0]) return;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int n = blockIdx.x * (blockDim.x >> 5) + warp;
+    const int n = (blockIdx.x * (blockDim.x >> 5) + warp) * (DUAL ? 1 : 2);
     if (n >= N) return;
     const int ex = tiles[3 * blockIdx.y], r0 = tiles[3 * blockIdx.y + 1], nr = tiles[3 * blockIdx.y + 2];
     const T* w1 = W + ((long long)ex * (DUAL ? 2 : 1) * N + n) * K;
-    const T* w2 = w1 + (long long)N * K;
+    const T* w2 = w1 + (DUAL ? (long long)N * K : (n + 1 < N ? (long long)K : 0));  // tail: re-read, never stored
     for (int m0 = 0; m0 < nr; m0 += MB) {
         const T* ar[MB];
 #pragma unroll
@@ -408,8 +410,7 @@ grouped_rows_kernel(const T* __restrict__ A, long long lda, const int* __restric
             const int kv = K / VEC;
             for (int v = lane; v < kv; v += 32) {
                 const uint4 wa = __ldcs(reinterpret_cast<const uint4*>(w1) + v);
-                uint4 wb = wa;
-                if (DUAL) wb = __ldcs(reinterpret_cast<const uint4*>(w2) + v);
+                const uint4 wb = __ldcs(reinterpret_cast<const uint4*>(w2) + v);
                 const T* pa = reinterpret_cast<const T*>(&wa);
                 const T* pb = reinterpret_cast<const T*>(&wb);
 #pragma unroll
@@ -421,7 +422,7 @@ grouped_rows_kernel(const T* __restrict__ A, long long lda, const int* __restric
                         for (int e = 0; e < VEC; ++e) {
                             const float xv = ldf(px + e);
                             acc[m] = fmaf(xv, ldf(pa + e), acc[m]);
-                            if (DUAL) acc2[m] = fmaf(xv, ldf(pb + e), acc2[m]);
+                            acc2[m] = fmaf(xv, ldf(pb + e), acc2[m]);
                         }
                     }
                 }
@@ -429,27 +430,28 @@ grouped_rows_kernel(const T* __restrict__ A, long long lda, const int* __restric
             k0 = kv * VEC;
         }
         for (int k = k0 + lane; k < K; k += 32) {
-            const float wa = ldf(w1 + k), wb = DUAL ? ldf(w2 + k) : 0.f;
+            const float wa = ldf(w1 + k), wb = ldf(w2 + k);
 #pragma unroll
             for (int m = 0; m < MB; ++m)
                 if (m0 + m < nr) {
                     const float xv = ldf(ar[m] + k);
                     acc[m] = fmaf(xv, wa, acc[m]);
-                    if (DUAL) acc2[m] = fmaf(xv, wb, acc2[m]);
+                    acc2[m] = fmaf(xv, wb, acc2[m]);
                 }
         }
 #pragma unroll
         for (int m = 0; m < MB; ++m) {
-            float y = warp_sum(acc[m]);
-            if (DUAL) {
-                const float u = warp_sum(acc2[m]);
-                y = y * sigmoidf_(y) * u;
-            }
+            float y = warp_sum(acc[m]), u = warp_sum(acc2[m]);
+            if (DUAL) y = y * sigmoidf_(y) * u;
             if (MODE == kRelu2) {
-                y = fmaxf(y, 0.f);
-                y *= y;
+                y = fmaxf(y, 0.f), u = fmaxf(u, 0.f);
+                y *= y, u *= u;
             }
-            if (lane == 0 && m0 + m < nr) stf(Cm + (long long)(r0 + m0 + m) * ldc + n, y);
+            if (lane == 0 && m0 + m < nr) {
+                TC* c = Cm + (long long)(r0 + m0 + m) * ldc + n;
+                stf(c, y);
+                if (!DUAL && n + 1 < N) stf(c + 1, u);
+            }
         }
     }
 }
@@ -539,6 +541,18 @@ extern "C" int llark_seq_moe_sort(const int* ids, int n_ent, int n_exp, int n_re
     return check_launch();
 }
 
+template <typename T, typename TC, int MODE>
+static void launch_rows(const T* A, long long lda, const int* perm, int top, const T* W, TC* C, const int* tiles,
+                        const int* meta, int max_tiles, int n_ent, int N, int K, int vec_ok, cudaStream_t st) {
+    const int per = MODE == kSiluGlu ? 8 : 16;  // output columns of a block's eight warps
+    const dim3 grid((N + per - 1) / per, max_tiles);
+    const int n_exp = max_tiles - (n_ent + kTileRows - 1) / kTileRows;
+    if (n_ent <= 8 * n_exp)  // a handful of rows per expert
+        grouped_rows_kernel<T, TC, MODE, 2><<<grid, 256, 0, st>>>(A, lda, perm, top, W, C, N, tiles, meta, N, K, vec_ok);
+    else
+        grouped_rows_kernel<T, TC, MODE, 8><<<grid, 256, 0, st>>>(A, lda, perm, top, W, C, N, tiles, meta, N, K, vec_ok);
+}
+
 template <typename T, int MODE>
 static int launch_up(const void* x, long long ldx, const int* perm, int top, const void* w, void* act, const int* tiles,
                      const int* meta, int max_tiles, int n_ent, int ff, int K, cudaStream_t st) {
@@ -546,8 +560,8 @@ static int launch_up(const void* x, long long ldx, const int* perm, int top, con
         const int vec = 16 / (int)sizeof(T);
         const int vec_ok = (K % vec == 0) && (ldx % vec == 0) &&
                            (((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w)) & 15) == 0);
-        grouped_rows_kernel<T, T, MODE><<<dim3((ff + 7) / 8, max_tiles), 256, 0, st>>>(
-            (const T*)x, ldx, perm, top, (const T*)w, (T*)act, ff, tiles, meta, ff, K, vec_ok);
+        launch_rows<T, T, MODE>((const T*)x, ldx, perm, top, (const T*)w, (T*)act, tiles, meta, max_tiles, n_ent, ff, K,
+                                vec_ok, st);
     } else {
         grouped_linear_kernel<T, T, MODE><<<dim3((ff + 63) / 64, max_tiles), 256, 0, st>>>(
             (const T*)x, ldx, perm, top, (const T*)w, (T*)act, ff, tiles, meta, ff, K);
@@ -573,18 +587,15 @@ extern "C" int llark_seq_moe_down(const void* act, const void* w_down, float* z,
                                   int max_tiles, int n_ent, int C, int ff, int act_fp32, cudaStream_t st) {
     if (max_tiles <= 0 || ff <= 0 || C <= 0 || !act || !w_down || !z || !tiles || !meta) return LLARK_EINVAL;
     if (n_ent <= kRowsRouteMaxEntries) {
-        dim3 g2((C + 7) / 8, max_tiles);
         const int esz = act_fp32 ? 4 : 2, vec = 16 / esz;
         const int vec_ok = (ff % vec == 0) &&
                            (((reinterpret_cast<uintptr_t>(act) | reinterpret_cast<uintptr_t>(w_down)) & 15) == 0);
         if (act_fp32)
-            grouped_rows_kernel<float, float, kPlain><<<g2, 256, 0, st>>>((const float*)act, ff, nullptr, 1,
-                                                                         (const float*)w_down, z, C, tiles, meta, C, ff,
-                                                                         vec_ok);
+            launch_rows<float, float, kPlain>((const float*)act, ff, nullptr, 1, (const float*)w_down, z, tiles, meta,
+                                              max_tiles, n_ent, C, ff, vec_ok, st);
         else
-            grouped_rows_kernel<bf16_t, float, kPlain><<<g2, 256, 0, st>>>((const bf16_t*)act, ff, nullptr, 1,
-                                                                          (const bf16_t*)w_down, z, C, tiles, meta, C, ff,
-                                                                          vec_ok);
+            launch_rows<bf16_t, float, kPlain>((const bf16_t*)act, ff, nullptr, 1, (const bf16_t*)w_down, z, tiles, meta,
+                                               max_tiles, n_ent, C, ff, vec_ok, st);
         return check_launch();
     }
     dim3 grid((C + 63) / 64, max_tiles);

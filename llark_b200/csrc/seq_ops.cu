@@ -1109,20 +1109,17 @@ static void launch_rows(const void* A, long long lda, const void* W, long long l
     const int vec_ok = (K % vec == 0) && (lda % vec == 0) && (ldw % vec == 0) &&
                        (((reinterpret_cast<uintptr_t>(A) | reinterpret_cast<uintptr_t>(W)) & 15) == 0);
     const int warps = 8;
-    // two columns per warp once that still leaves several warps per SM (148 SMs); one for narrow outputs
-    const bool two = (long long)N >= 2LL * warps * 148 * 2 || act == LLARK_ACT_RELU_GLU;  // (a gate and its up column)
+    // one or two rows: two columns per warp once that still leaves several warps per SM (148 SMs), one for narrow outputs.
+    // More rows: blocks of two rows and always two columns (the later row blocks read the weights from L2; a wider row block
+    // costs more in registers, and so in warps, than it saves)
+    const bool two = M > 2 || (long long)N >= 2LL * warps * 148 * 2 || act == LLARK_ACT_RELU_GLU;  // (a gate and its up column)
     const int nc = two ? 2 : 1;
     const unsigned gx = (unsigned)((N + warps * nc - 1) / (warps * nc));
 #define LLARK_ROWS(MB_, NC_)                                                                                            \
     linear_rows_kernel<T, TC, MB_, NC_><<<dim3(gx, (M + MB_ - 1) / MB_), warps * 32, 0, st>>>(                          \
         (const T*)A, lda, (const T*)W, ldw, (TC*)C, ldc, bias, M, N, K, vec_ok, act)
-    if (M <= 2) {
-        if (two) LLARK_ROWS(2, 2);
-        else LLARK_ROWS(2, 1);
-    } else {
-        if (two) LLARK_ROWS(8, 2);
-        else LLARK_ROWS(8, 1);
-    }
+    if (two) LLARK_ROWS(2, 2);
+    else LLARK_ROWS(2, 1);
 #undef LLARK_ROWS
 }
 

@@ -484,6 +484,15 @@ def _actf(dtype):
 # of the weight matrix); above it the tcgen05 GEMM core (bf16, at least one 64-wide tile in N and K, rows that TMA can
 # address) or the tiled SIMT kernel (fp32 mode, small or odd shapes)
 LINEAR_ROWS_MAX = 8
+
+
+def linear_rows_pays(M, N, K):
+    """Whether the weight-streaming kernel beats the tcgen05 core at M <= LINEAR_ROWS_MAX rows. Two rows ride on one read of a
+    weight; beyond that its FMAs grow with M N K, while the core takes a fixed time plus one that grows with K (measured on a
+    B200: rows 8 us + M N K / 4.1e6 us, core 16 us + K / 220 us, the launch included)."""
+    return M <= 2 or M * N * K < 32500000 + 18300 * K
+
+
 LINEAR_STATS = {"rows": 0, "tcgen05": 0, "simt": 0}
 
 
@@ -511,12 +520,15 @@ def linear(a, w, bias=None, out_dtype=None, out=None, act=None):
     if bias is not None:
         _req(bias, torch.float32)
     vec = 4 if c_fp32 else 8
-    if M <= LINEAR_ROWS_MAX:
+    rows = M <= LINEAR_ROWS_MAX and (in_fp32 or linear_rows_pays(M, N, K))
+    tc = (not rows and not in_fp32 and not (c_fp32 and act == "relu_glu") and K >= 64 and N >= 64 and K % 8 == 0 and a.stride(0) % 8 == 0
+          and w.stride(0) % 8 == 0 and out.stride(0) % vec == 0 and a.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0
+          and out.data_ptr() % 16 == 0)
+    if rows or (M <= LINEAR_ROWS_MAX and not tc):
         LINEAR_STATS["rows"] += 1
         check(lib().llark_linear_rows(_p(a), a.stride(0), _p(w), w.stride(0), _p(out), out.stride(0), c_fp32, _p(bias),
                                       M, N, K, in_fp32, code, _stream()), "linear_rows")
-    elif (not in_fp32 and not (c_fp32 and act == "relu_glu") and K >= 64 and N >= 64 and K % 8 == 0 and a.stride(0) % 8 == 0 and w.stride(0) % 8 == 0 and out.stride(0) % vec == 0
-          and a.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0 and out.data_ptr() % 16 == 0):
+    elif tc:
         LINEAR_STATS["tcgen05"] += 1
         gemm(a, w, bias=bias, out=out, M=M, N=N, K=K, act=act)
     else:

@@ -480,8 +480,8 @@ def _actf(dtype):
     return int(dtype == torch.float32)
 
 
-# rows up to which a linear is the weight-streaming kernel (the activations then sit in L1 / L2, the op is a pure read
-# of the weight matrix); above it the tcgen05 GEMM core (bf16, at least one 64-wide tile in N and K, rows that TMA can
+# rows up to which a linear can be the weight-streaming kernel (the activations then sit in L1 / L2, the op is a pure read
+# of the weight matrix; linear_rows_pays says when it is); otherwise the tcgen05 GEMM core (bf16, at least one 64-wide tile in N and K, rows that TMA can
 # address) or the tiled SIMT kernel (fp32 mode, small or odd shapes)
 LINEAR_ROWS_MAX = 8
 
@@ -494,8 +494,6 @@ def linear_rows_pays(M, N, K):
 
 
 LINEAR_STATS = {"rows": 0, "tcgen05": 0, "simt": 0}
-
-
 LINEAR_ACTS = {None: 0, "relu2": 1, "relu_glu": 2}
 
 

@@ -57,19 +57,22 @@ int llark_gemm(const void* A, int a_mn_major, long long lda, const void* B, int 
  * Results are bit-identical to the unfused sequences (same bf16 rounding points).
  *   LLARK_EPI_RELU2       C = relu(acc + bias)^2, rounded once
  *   LLARK_EPI_RELU_GLU    the rows of B alternate gate, up: C bf16 [M, N / 2], C[:, c] = relu(z[:, 2c]) * z[:, 2c + 1] with
- *                         z = acc + bias, rounded once */
+ *                         z = acc + bias, rounded once
+ *   LLARK_EPI_CLAMP_GLU   the same with C[:, c] = g * sigmoid(f1 * g) * (u + 1), g = min(z[:, 2c], f0), u = z[:, 2c + 1]
+ *                         clamped to -f0 .. f0 */
 /*   LLARK_EPI_SEGMENTS    not an epilogue: the rows of A / C come in runs that each multiply their own block of B (stacked
  *                         [i1, N, K]); a = device int triples (block, first row, rows <= 256), i0 = their number (an upper
- *                         bound when b points at a device word with the real number), ld = LLARK_EPI_NONE or
- *                         LLARK_EPI_RELU2. Used by llark_gemm_segments. */
+ *                         bound when b points at a device word with the real number), ld = LLARK_EPI_NONE,
+ *                         LLARK_EPI_RELU2 or LLARK_EPI_CLAMP_GLU. Used by llark_gemm_segments. */
 enum { LLARK_EPI_NONE = 0, LLARK_EPI_QUICK_GELU = 1, LLARK_EPI_ROPE = 2, LLARK_EPI_SWIGLU_BWD = 3, LLARK_EPI_SEGMENTS = 4,
-       LLARK_EPI_RELU2 = 5, LLARK_EPI_RELU_GLU = 6 };
+       LLARK_EPI_RELU2 = 5, LLARK_EPI_RELU_GLU = 6, LLARK_EPI_CLAMP_GLU = 7 };
 typedef struct LlarkGemmEpilogue {
     int kind;
     const void* a;
     const void* b;
     long long ld;
     int i0, i1;
+    float f0, f1;
 } LlarkGemmEpilogue;
 int llark_gemm_ex(const void* A, int a_mn_major, long long lda, const void* B, int b_mn_major, long long ldb, void* C,
                   long long ldc, int c_fp32, const void* bias, int bias_fp32, const void* R, long long ldr, int M, int N,
@@ -282,7 +285,8 @@ int llark_v32_ce_fwd(const float* logits, long long ldv, int V, const long long*
  * state store. The residual stream, norms, scores, softmax and recurrent state are fp32; `act_fp32` selects the
  * activation / matrix dtype (0: bf16, 1: float = the all-fp32 mode). */
 int llark_seq_embed(const int* ids, const int* tok_seq, const int* cu, const int* pos0, const void* table,
-                    const void* pos_table, float scale, float* x, int n_tok, int C, int act_fp32, cudaStream_t stream);
+                    const void* pos_table, float scale, float* x, void* x_act, int n_tok, int C, int act_fp32,
+                    cudaStream_t stream); /* x_act (optional): a copy of x in the activation dtype */
 /* y = h + conv(h): causal depthwise convolution over time, w fp32 [C, taps], tail fp32 [slots, taps-1, C] = the last
  * taps-1 inputs of each request, oldest first. inline_tail = 1 (every request brings one token) also shifts the tail;
  * otherwise call llark_seq_conv_tail after it. */
@@ -303,6 +307,13 @@ int llark_seq_gated_norm_add(const float* x, const float* y, const float* gate, 
 int llark_seq_rmsnorm_rows(const float* x, const int* rows, const float* w, void* out, int n_rows, int C, float eps,
                            int act_fp32, cudaStream_t stream);
 int llark_seq_relu2(const void* u, void* y, long long n, int act_fp32, cudaStream_t stream);
+/* Layer norm (mean off, / sqrt(mean squared deviation + eps), times a weight) around a residual sum: f = y (optional) + sum_{k <
+ * top} wts[t, k] * z[pos_of[t * top + k]] (wts NULL: 1); o = x + norm(f) * w_post (w_post NULL: x + f) -> x_out (optional);
+ * norm(o) * w_next (w_next NULL: o) -> x_act (optional, activation dtype). Without y and z: o = x, and rows (optional) names
+ * the rows of x. */
+int llark_seq_layer_norm_add(const float* x, const int* rows, const float* y, const float* z, const int* pos_of,
+                             const float* wts, int top, const float* w_post, const float* w_next, float* x_out, void* x_act,
+                             long long n_rows, int C, float eps, int act_fp32, cudaStream_t stream);
 /* out[i] = tanh(alpha * x[rows[i]]) * w + b in the activation dtype (rows == NULL: row i). */
 int llark_seq_tanh_norm(const float* x, const int* rows, float alpha, const float* w, const float* b, void* out, int n_rows,
                         int C, int out_fp32, cudaStream_t stream);
@@ -315,12 +326,15 @@ int llark_seq_tanh_norm_add(const float* x, const float* y, const float* z, cons
 /* C[M,N] = act(A[M,K] W[N,K]^T (+ bias fp32[N])), fp32 accumulation, A / W bf16 or (in_fp32) float, C float if c_fp32.
  * _rows: weight-streaming, for a handful of rows (decode). _simt: tiled, any shape, true fp32 when in_fp32.
  * act: LLARK_ACT_RELU2 = relu(z)^2; LLARK_ACT_RELU_GLU = the rows of W alternate gate, up and C [M, N / 2] gets
- * relu(z[:, 2c]) * z[:, 2c + 1]. */
-enum { LLARK_ACT_NONE = 0, LLARK_ACT_RELU2 = 1, LLARK_ACT_RELU_GLU = 2 };
+ * relu(z[:, 2c]) * z[:, 2c + 1]; LLARK_ACT_CLAMP_GLU = the same with g * sigmoid(act_slope * g) * (u + 1), g = min(z[:, 2c],
+ * act_limit), u = z[:, 2c + 1] clamped to -act_limit .. act_limit. */
+enum { LLARK_ACT_NONE = 0, LLARK_ACT_RELU2 = 1, LLARK_ACT_RELU_GLU = 2, LLARK_ACT_CLAMP_GLU = 3 };
 int llark_linear_rows(const void* A, long long lda, const void* W, long long ldw, void* C, long long ldc, int c_fp32,
-                      const float* bias, int M, int N, int K, int in_fp32, int act, cudaStream_t stream);
+                      const float* bias, int M, int N, int K, int in_fp32, int act, float act_limit, float act_slope,
+                      cudaStream_t stream);
 int llark_linear_simt(const void* A, long long lda, const void* W, long long ldw, void* C, long long ldc, int c_fp32,
-                      const float* bias, int M, int N, int K, int in_fp32, int act, cudaStream_t stream);
+                      const float* bias, int M, int N, int K, int in_fp32, int act, float act_limit, float act_slope,
+                      cudaStream_t stream);
 /* Per-head RMS norm of the q (H heads at column q_off) and k (G heads at k_off) parts of src fp32 [n_tok, ld] with
  * weights wq, wk fp32 [D]: qn [n_tok, H, D], kn [n_tok, G, D], vraw = the un-normed k. kring / vring non-NULL: also
  * written to ring entry position % cap of the request's slot (only when every request brings one token). */
@@ -355,12 +369,13 @@ int llark_seq_qkv_rotary(const float* src, long long ld, int q_off, int k_off, i
  * sees j <= i with floor(j / chunk) = floor(i / chunk). softcap > 0: score <- softcap * tanh(score / softcap). vfreq fp32
  * [E / 2] (optional): the values are stored rotated by their own position (llark_seq_qkv_rotary); each head's weighted sum is
  * turned back by the query's position before the gate (v_interleaved: pairs (2m, 2m + 1), else (m, m + E/2)).
- * out [n_tok, H, E]. */
+ * out: H * E columns times out_scale, rows out_ld apart. */
 int llark_seq_swa_attn(const void* qn, const void* kn, const void* vv, const void* kring, const void* vring,
                        const float* gate, long long gate_ld, const float* scale_h, void* out, const int* tok_seq,
                        const int* cu, const int* pos0, const int* slot, int n_tok, int H, int G, int D, int E, int window,
                        int cap, int from_ring_only, const float* sink, int gate_per_head, int chunk, float softcap,
-                       const float* vfreq, int v_interleaved, int act_fp32, cudaStream_t stream);
+                       const float* vfreq, int v_interleaved, long long out_ld, float out_scale, int act_fp32,
+                       cudaStream_t stream);
 /* The same attention for steps that bring many tokens per request (prompts, portions): bf16 only, D = E a multiple of
  * 16 up to 256, 64-query CTAs on mma.sync with fp32 scores / softmax (csrc/seq_swa_mma.cu). max_len = the longest
  * request of the step. Un-rotation in halves needs D = 64, 128 or 256. */
@@ -368,7 +383,7 @@ int llark_seq_swa_attn_mma(const void* qn, const void* kn, const void* vv, const
                            const float* gate, long long gate_ld, const float* scale_h, void* out, const int* cu,
                            const int* pos0, const int* slot, int n_seq, int max_len, int H, int G, int D, int window,
                            int cap, const float* sink, int gate_per_head, int chunk, float softcap, const float* vfreq,
-                           int v_interleaved, cudaStream_t stream);
+                           int v_interleaved, long long out_ld, float out_scale, cudaStream_t stream);
 int llark_seq_kv_ring_write(const void* kn, const void* vv, void* kring, void* vring, const int* tok_seq, const int* cu,
                             const int* pos0, const int* slot, int n_tok, int GD, int GE, int cap, int act_fp32,
                             cudaStream_t stream);
@@ -389,6 +404,27 @@ int llark_seq_glr_combine(const float* state, float* chunk_state, const float* c
                           const int* slot, int n_seq, int H, int D, int E, cudaStream_t stream);
 int llark_seq_head_rmsnorm(const float* x, const float* w, void* out, long long n_rows, int E, float eps, int act_fp32,
                            cudaStream_t stream);
+
+/* Linear attention with a fixed decay per head (csrc/seq_decay.cu): S_t = decay_h S_(t-1) + k_t v_t^T, o_t = S_t^T q_t, all
+ * fp32. q and k ([H, D] at q_off, k_off) and v ([H, E] at v_off) are columns of src; n_rot > 0: the first n_rot entries of q
+ * and k heads are rotated (pairs (i, i + n_rot / 2), interleaved: (2i, 2i + 1)) by the angles whose (cos, sin) row t of cs
+ * holds (llark_seq_rotary_table); k is multiplied by k_scale; silu: q, k and v pass through SiLU (without rotation).
+ * pow_h [H, pow_ld]: decay_h^0, decay_h^1, ... Work items and their states as in llark_seq_glr_scan.
+ * _rows: token by token, D <= 1024, max_n = the longest item. _chunks: 32 tokens at a time as split TF32 products (fp32
+ * accuracy), D <= 128, pow_ld >= 33, o may be NULL (states only). _combine: chunk_state[w] (what item w builds from zero)
+ * becomes the state item w starts from; pow_ld > the longest item. */
+int llark_seq_rotary_table(const float* freq, int n_freq, const int* tok_seq, const int* cu, const int* pos0, float* cs,
+                           int n_tok, cudaStream_t stream);
+int llark_seq_decay_rows(const float* src, long long ld, int q_off, int k_off, int v_off, const float* cs, int n_rot,
+                         int interleaved, float k_scale, int silu, const float* pow_h, int pow_ld, const float* init_buf,
+                         float* final_buf, float* o, const int* item_row0, const int* item_n, const int* item_init,
+                         const int* item_final, int n_items, int max_n, int H, int D, int E, cudaStream_t stream);
+int llark_seq_decay_chunks(const float* src, long long ld, int q_off, int k_off, int v_off, const float* cs, int n_rot,
+                           int interleaved, float k_scale, int silu, const float* pow_h, int pow_ld, const float* init_buf,
+                           float* final_buf, float* o, const int* item_row0, const int* item_n, const int* item_init,
+                           const int* item_final, int n_items, int H, int D, int E, cudaStream_t stream);
+int llark_seq_decay_combine(const float* state, float* chunk_state, const float* pow_h, int pow_ld, const int* item_n,
+                            const int* seq_item0, const int* slot, int n_seq, int H, int D, int E, cudaStream_t stream);
 
 /* ---- further parts of layer-list decoders: grouped RMS norm, parallel-sublayer residual, delta-rule recurrences
  * (csrc/seq_delta.cu), latent attention (csrc/seq_latent.cu), routed mixture of experts (csrc/seq_moe.cu) ---- */
@@ -418,10 +454,10 @@ int llark_seq_delta_prep(int rule, const float* q, long long q_ld, const float* 
  * correct = 0: the p1 term is skipped (rules whose p1 is zero) */
 int llark_seq_delta_scan(const float* vec, const float* v, long long v_ld, float* state, float* o, const int* cu,
                          const int* slot, int n_seq, int n_tok, int H, int D, int E, int correct, cudaStream_t stream);
-/* per-head RMS norm of x fp32 [n_tok, H, E], times w ([E] shared or [H, E]), times sigmoid(gate) (gate_silu: times
- * gate * sigmoid(gate)) -> ACT */
+/* per-head RMS norm of x fp32 [n_tok, H, E], times w ([E] shared or [H, E]; optional), times sigmoid(gate) (gate_silu: times
+ * gate * sigmoid(gate)) -> ACT, rows out_ld apart */
 int llark_seq_head_norm_gate(const float* x, const float* w, int w_per_head, const float* gate, long long gate_ld,
-                             void* out, long long n_tok, int H, int E, float eps, int gate_silu, int act_fp32,
+                             void* out, long long out_ld, long long n_tok, int H, int E, float eps, int gate_silu, int act_fp32,
                              cudaStream_t stream);
 /* read-out of a state-space mixer: y = (o + skip[h] * xin) * silu(gate) over the H * E inner channels, RMS norm of each
  * of `groups` equal consecutive parts, times w fp32 [H * E] -> ACT [n_tok, H * E] */
@@ -454,10 +490,10 @@ int llark_seq_head_linear(const void* x, int x_fp32, long long ldx, int x_hs, co
 /* y = tanh(u), fp32 in, ACT out */
 int llark_seq_tanh(const float* u, void* y, long long n, int act_fp32, cudaStream_t stream);
 /* C[off[e] .. off[e+1]) = A[same rows] @ B[e]^T, e < n_seg; B bf16 [n_seg, N, K]; seg_off_host on the host; epi:
- * LLARK_EPI_NONE or LLARK_EPI_RELU2 */
+ * LLARK_EPI_NONE, LLARK_EPI_RELU2 or LLARK_EPI_CLAMP_GLU (limit f0, slope f1) */
 int llark_gemm_segments(const void* A, long long lda, const void* B, void* C, long long ldc, int c_fp32,
                         const int* seg_off_host, int n_seg, const int* seg_tiles_dev, int n_tiles, const int* seg_count_dev,
-                        int m_total, int N, int K, int epi, cudaStream_t stream);
+                        int m_total, int N, int K, int epi, float f0, float f1, cudaStream_t stream);
 /* routed mixture of experts (see csrc/seq_moe.cu) */
 int llark_seq_moe_route(const float* logits, long long ld, int* ids, float* wts, int n_tok, int n_exp, int n_groups,
                         int keep, int top, float scale, cudaStream_t stream);
@@ -465,21 +501,24 @@ int llark_seq_moe_route(const float* logits, long long ld, int* ids, float* wts,
  * weights = the chosen experts' plain scores * scale */
 int llark_seq_moe_route_bias(const float* logits, long long ld, const float* correction, int* ids, float* wts, int n_tok,
                              int n_exp, int n_groups, int keep, int top, float scale, cudaStream_t stream);
-/* the `top` largest logits of each row; weights = softmax over those logits */
+/* the `top` largest logits of each row; weights = softmax over those logits, or, sigmoid_wts, the sigmoid of each */
 int llark_seq_moe_route_top(const float* logits, long long ld, int* ids, float* wts, int n_tok, int n_exp, int top,
-                            cudaStream_t stream);
+                            int sigmoid_wts, cudaStream_t stream);
 int llark_seq_moe_tile_rows(void);
 /* meta[0] = number of 64-row tiles; with tiles256: 256-row tiles for llark_gemm_segments, their number in meta[1];
  * experts >= n_real have no weights and get no tiles */
 int llark_seq_moe_sort(const int* ids, int n_ent, int n_exp, int n_real, int* perm, int* pos_of, int* tiles, int* meta,
                        int* seg_off, int* tiles256, cudaStream_t stream);
-/* xs[p] = x[perm[p] / top] (rows in sorted order); act = silu(gu[:, :ff]) * gu[:, ff:] */
-int llark_seq_moe_gather(const void* x, long long ldx, const int* perm, int top, void* xs, int n_ent, int C, int act_fp32,
-                         cudaStream_t stream);
+/* xs[p] = x[perm[p] / top] (rows in sorted order; times in_wts[perm[p]] when given); act = silu(gu[:, :ff]) * gu[:, ff:] */
+int llark_seq_moe_gather(const void* x, long long ldx, const int* perm, int top, void* xs, int n_ent, int C,
+                         const float* in_wts, int act_fp32, cudaStream_t stream);
 int llark_seq_silu_mul(const void* gu, void* act, long long rows, int ff, int act_fp32, cudaStream_t stream);
-/* act[p] = silu(gate x) * (up x) with w [n, 2 * ff, K] (gated), or relu(w x)^2 with w [n, ff, K]; x = row perm[p] / top */
+/* act[p] = silu(gate x) * (up x) with w [n, 2 * ff, K] (gated = 1), relu(w x)^2 with w [n, ff, K] (gated = 0), or the clamped
+ * gated unit of LLARK_ACT_CLAMP_GLU with w [n, 2 * ff, K], gate and up rows alternating (gated = 2); x = row perm[p] / top
+ * times in_wts[perm[p]] when given */
 int llark_seq_moe_up(const void* x, long long ldx, const int* perm, int top, const void* w, void* act, const int* tiles,
-                     const int* meta, int max_tiles, int n_ent, int ff, int K, int gated, int act_fp32, cudaStream_t stream);
+                     const int* meta, int max_tiles, int n_ent, int ff, int K, int gated, const float* in_wts, float limit,
+                     float slope, int act_fp32, cudaStream_t stream);
 int llark_seq_moe_down(const void* act, const void* w_down, float* z, const int* tiles, const int* meta, int max_tiles,
                        int n_ent, int C, int ff, int act_fp32, cudaStream_t stream);
 

@@ -27,7 +27,8 @@ SEQ_SYMBOLS = [
     "llark_seq_moe_down", "llark_seq_tanh", "llark_seq_moe_gather", "llark_seq_silu_mul",
     "llark_seq_qkv_headnorm", "llark_seq_skip_gate_group_norm", "llark_seq_post_norm", "llark_seq_glu_clamped",
     "llark_seq_logit_cap", "llark_seq_moe_route_bias", "llark_seq_qkv_rotary", "llark_seq_gated_norm_add",
-    "llark_seq_tanh_norm", "llark_seq_tanh_norm_add", "llark_seq_moe_route_top",
+    "llark_seq_tanh_norm", "llark_seq_tanh_norm_add", "llark_seq_moe_route_top", "llark_seq_layer_norm_add",
+    "llark_seq_rotary_table", "llark_seq_decay_rows", "llark_seq_decay_chunks", "llark_seq_decay_combine",
 ]
 # what libllark_serve.so (`make serve`: GEMM core + decode linears + the ops above) exports
 SERVE_SYMBOLS = SEQ_SYMBOLS + ["llark_last_cuda_error", "llark_init", "llark_gemm", "llark_gemm_ex", "llark_gemv",
@@ -54,10 +55,10 @@ _lib = None
 class GemmEpilogue(ctypes.Structure):
     """LlarkGemmEpilogue of include/llark_b200.h."""
     _fields_ = [("kind", ctypes.c_int), ("a", ctypes.c_void_p), ("b", ctypes.c_void_p), ("ld", ctypes.c_longlong),
-                ("i0", ctypes.c_int), ("i1", ctypes.c_int)]
+                ("i0", ctypes.c_int), ("i1", ctypes.c_int), ("f0", ctypes.c_float), ("f1", ctypes.c_float)]
 
 
-EPI_NONE, EPI_QUICK_GELU, EPI_ROPE, EPI_SWIGLU_BWD, EPI_RELU2, EPI_RELU_GLU = 0, 1, 2, 3, 5, 6
+EPI_NONE, EPI_QUICK_GELU, EPI_ROPE, EPI_SWIGLU_BWD, EPI_RELU2, EPI_RELU_GLU, EPI_CLAMP_GLU = 0, 1, 2, 3, 5, 6, 7
 
 
 class LlarkError(RuntimeError):
@@ -143,24 +144,29 @@ def lib():
             "llark_v32_swiglu_fwd": ([P, P, LL, I, P], I),
             "llark_v32_attn_fwd": ([P, P, P, I, I, I, I, F, P], I),
             "llark_v32_ce_fwd": ([P, LL, I, P, I, I, P, P, P], I),
-            "llark_seq_embed": ([P, P, P, P, P, P, F, P, I, I, I, P], I),
+            "llark_seq_embed": ([P, P, P, P, P, P, F, P, P, I, I, I, P], I),
             "llark_seq_short_conv": ([P, P, P, P, P, P, P, I, I, I, I, I, P], I),
             "llark_seq_conv_tail": ([P, P, P, P, I, I, I, P], I),
             "llark_seq_add_rmsnorm": ([P, P, P, P, P, LL, I, F, I, P], I),
             "llark_seq_rmsnorm_rows": ([P, P, P, P, I, I, F, I, P], I),
             "llark_seq_relu2": ([P, P, LL, I, P], I),
-            "llark_linear_rows": ([P, LL, P, LL, P, LL, I, P, I, I, I, I, I, P], I),
-            "llark_linear_simt": ([P, LL, P, LL, P, LL, I, P, I, I, I, I, I, P], I),
+            "llark_linear_rows": ([P, LL, P, LL, P, LL, I, P, I, I, I, I, I, F, F, P], I),
+            "llark_linear_simt": ([P, LL, P, LL, P, LL, I, P, I, I, I, I, I, F, F, P], I),
             "llark_seq_qk_headnorm": ([P, LL, I, I, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, F, I, P], I),
             "llark_seq_qkv_headnorm": ([P, LL, I, I, I, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, F, I, I, P], I),
-            "llark_seq_swa_attn": ([P, P, P, P, P, P, LL, P, P, P, P, P, P, I, I, I, I, I, I, I, I, P, I, I, F, P, I, I, P], I),
-            "llark_seq_swa_attn_mma": ([P, P, P, P, P, P, LL, P, P, P, P, P, I, I, I, I, I, I, I, P, I, I, F, P, I, P], I),
+            "llark_seq_swa_attn": ([P, P, P, P, P, P, LL, P, P, P, P, P, P, I, I, I, I, I, I, I, I, P, I, I, F, P, I, LL, F, I, P], I),
+            "llark_seq_swa_attn_mma": ([P, P, P, P, P, P, LL, P, P, P, P, P, I, I, I, I, I, I, I, P, I, I, F, P, I, LL, F, P], I),
             "llark_seq_qkv_rotary": ([P, LL, I, I, I, P, P, P, I, I, P, I, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, I, I,
                                       P], I),
             "llark_seq_gated_norm_add": ([P, P, P, LL, P, P, P, P, LL, I, F, I, P], I),
             "llark_seq_tanh_norm": ([P, P, F, P, P, P, I, I, I, P], I),
             "llark_seq_tanh_norm_add": ([P, P, P, P, P, I, F, P, P, F, P, P, P, P, LL, I, I, P], I),
-            "llark_seq_moe_route_top": ([P, LL, P, P, I, I, I, P], I),
+            "llark_seq_moe_route_top": ([P, LL, P, P, I, I, I, I, P], I),
+            "llark_seq_layer_norm_add": ([P, P, P, P, P, P, I, P, P, P, P, LL, I, F, I, P], I),
+            "llark_seq_rotary_table": ([P, I, P, P, P, P, I, P], I),
+            "llark_seq_decay_rows": ([P, LL, I, I, I, P, I, I, F, I, P, I, P, P, P, P, P, P, P, I, I, I, I, I, P], I),
+            "llark_seq_decay_chunks": ([P, LL, I, I, I, P, I, I, F, I, P, I, P, P, P, P, P, P, P, I, I, I, I, P], I),
+            "llark_seq_decay_combine": ([P, P, P, I, P, P, P, I, I, I, I, P], I),
             "llark_seq_kv_ring_write": ([P, P, P, P, P, P, P, P, I, I, I, I, I, P], I),
             "llark_seq_glr_scan": ([P, LL, I, I, I, P, P, P, P, P, P, P, P, P, I, I, I, I, P], I),
             "llark_seq_glr_combine": ([P, P, P, P, P, I, I, I, I, P], I),
@@ -171,7 +177,7 @@ def lib():
             "llark_seq_conv_act": ([P, LL, P, P, P, P, P, P, I, I, I, I, I, P, P], I),
             "llark_seq_delta_prep": ([I, P, LL, P, LL, P, LL, P, P, P, LL, P, I, I, I, I, F, P], I),
             "llark_seq_delta_scan": ([P, P, LL, P, P, P, P, I, I, I, I, I, I, P], I),
-            "llark_seq_head_norm_gate": ([P, P, I, P, LL, P, LL, I, I, F, I, I, P], I),
+            "llark_seq_head_norm_gate": ([P, P, I, P, LL, P, LL, LL, I, I, F, I, I, P], I),
             "llark_seq_skip_gate_group_norm": ([P, P, LL, P, P, LL, P, P, LL, I, I, I, F, I, P], I),
             "llark_seq_post_norm": ([P, F, P, P, P, P, F, P, P, P, P, I, I, P, P, P, LL, I, F, I, P], I),
             "llark_seq_glu_clamped": ([P, P, LL, I, F, F, I, P], I),
@@ -182,11 +188,11 @@ def lib():
             "llark_seq_moe_route": ([P, LL, P, P, I, I, I, I, I, F, P], I),
             "llark_seq_moe_tile_rows": ([], I),
             "llark_seq_moe_sort": ([P, I, I, I, P, P, P, P, P, P, P], I),
-            "llark_seq_moe_gather": ([P, LL, P, I, P, I, I, I, P], I),
+            "llark_seq_moe_gather": ([P, LL, P, I, P, I, I, P, I, P], I),
             "llark_seq_silu_mul": ([P, P, LL, I, I, P], I),
-            "llark_seq_moe_up": ([P, LL, P, I, P, P, P, P, I, I, I, I, I, I, P], I),
+            "llark_seq_moe_up": ([P, LL, P, I, P, P, P, P, I, I, I, I, I, P, F, F, I, P], I),
             "llark_seq_moe_down": ([P, P, P, P, P, I, I, I, I, I, P], I),
-            "llark_gemm_segments": ([P, LL, P, P, LL, I, P, I, P, I, P, I, I, I, I, P], I),
+            "llark_gemm_segments": ([P, LL, P, P, LL, I, P, I, P, I, P, I, I, I, I, F, F, P], I),
             "llark_seq_tanh": ([P, P, LL, I, P], I),
         }
         for name, (argtypes, restype) in sig.items():

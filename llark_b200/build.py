@@ -20,7 +20,7 @@ def _sources_newer_than(lib, names):
 
 
 SERVE_SOURCES = ("gemm_tcgen05.cu", "gemv.cu", "seq_ops.cu", "seq_mixers.cu", "seq_swa_mma.cu", "seq_delta.cu",
-                 "seq_latent.cu", "seq_moe.cu", "common.cuh")
+                 "seq_latent.cu", "seq_moe.cu", "seq_decay.cu", "common.cuh")
 
 
 def ensure_built(verbose=False):

@@ -69,6 +69,7 @@ struct GemmParams {
     const void* epi_b;
     long long epi_ld;
     int epi_i0, epi_i1;
+    float epi_f0, epi_f1;
     // rows-in-runs mode (CTA-pair kernel, K-major bf16 operands): m-block i covers rows seg_tiles[3i+1] .. + seg_tiles[3i+2]
     // of A / C and multiplies weight block seg_tiles[3i] of B (stacked [blocks, N, K]); nullptr: one matrix
     const int* seg_tiles;
@@ -167,12 +168,19 @@ __device__ __forceinline__ void epilogue_store_chunk(const GemmParams& p, long l
                 const float r = fmaxf(f[e], 0.f);
                 f[e] = r * r;
             }
-        } else if constexpr (EPI == 6) {
+        } else if constexpr (EPI == 6 || EPI == 7) {
             // gate / up columns alternate (N even, C bf16): four results per eight columns
             __nv_bfloat16* cptr = reinterpret_cast<__nv_bfloat16*>(p.C) + row * p.ldc + (col >> 1);
             float g[4];
 #pragma unroll
-            for (int e = 0; e < 4; ++e) g[e] = fmaxf(f[2 * e], 0.f) * f[2 * e + 1];
+            for (int e = 0; e < 4; ++e) {
+                if constexpr (EPI == 6) {
+                    g[e] = fmaxf(f[2 * e], 0.f) * f[2 * e + 1];
+                } else {
+                    const float gv = fminf(f[2 * e], p.epi_f0), uv = fminf(fmaxf(f[2 * e + 1], -p.epi_f0), p.epi_f0);
+                    g[e] = __fdividef(gv, 1.f + __expf(-p.epi_f1 * gv)) * (uv + 1.f);
+                }
+            }
             if (full8) {
                 *reinterpret_cast<uint2*>(cptr) = make_uint2(pack_bf16x2(g[0], g[1]), pack_bf16x2(g[2], g[3]));
             } else {
@@ -501,7 +509,7 @@ __device__ __forceinline__ void epi_staged_bf16(const GemmParams& p, long long r
 template <int EPI>
 __device__ __forceinline__ void epilogue_dispatch(const GemmParams& p, long long row0, long long m_end, int lane, int ncol0,
                                                   uint32_t taddr, float* stg) {
-    if ((EPI == 2 && ncol0 < p.epi_i1) || EPI == 5 || EPI == 6 || !p.staged) {
+    if ((EPI == 2 && ncol0 < p.epi_i1) || EPI == 5 || EPI == 6 || EPI == 7 || !p.staged) {
         const long long row = row0 + lane;
         epilogue_tile<EPI>(p, row, row < m_end, ncol0, taddr);
         return;
@@ -1202,8 +1210,9 @@ extern "C" int llark_gemm_ex(const void* A, int a_mn_major, long long lda, const
     if (M <= 0 || N <= 0 || K <= 0 || !A || !B || !C) return LLARK_EINVAL;
     const bool segs = ep && ep->kind == LLARK_EPI_SEGMENTS;
     if (segs) {
-        // a = device tile list, i0 = its length, i1 = weight blocks stacked in B; ld = LLARK_EPI_NONE or LLARK_EPI_RELU2
-        if ((ep->ld != LLARK_EPI_NONE && ep->ld != LLARK_EPI_RELU2) || !ep->a || ep->i0 <= 0 || ep->i1 <= 0 || a_mn_major || b_mn_major || in_fp32 || bias || R ||
+        // a = device tile list, i0 = its length, i1 = weight blocks stacked in B; ld = the epilogue of the product
+        if ((ep->ld != LLARK_EPI_NONE && ep->ld != LLARK_EPI_RELU2 && ep->ld != LLARK_EPI_CLAMP_GLU) ||
+            (ep->ld == LLARK_EPI_CLAMP_GLU && (c_fp32 || (N % 2) || ldc < N / 2)) || !ep->a || ep->i0 <= 0 || ep->i1 <= 0 || a_mn_major || b_mn_major || in_fp32 || bias || R ||
             !llark_gemm_get_mode())
             return LLARK_EINVAL;
     } else if (ep && ep->kind != LLARK_EPI_NONE) {
@@ -1227,6 +1236,7 @@ extern "C" int llark_gemm_ex(const void* A, int a_mn_major, long long lda, const
                 if (R || a_mn_major || b_mn_major || in_fp32) return LLARK_EINVAL;
                 break;
             case LLARK_EPI_RELU_GLU:
+            case LLARK_EPI_CLAMP_GLU:
                 if (R || a_mn_major || b_mn_major || in_fp32 || c_fp32 || (N % 2) || ldc < N / 2) return LLARK_EINVAL;
                 break;
             default:
@@ -1339,6 +1349,8 @@ extern "C" int llark_gemm_ex(const void* A, int a_mn_major, long long lda, const
     p.epi_ld = ep ? ep->ld : 0;
     p.epi_i0 = ep ? ep->i0 : 0;
     p.epi_i1 = ep ? ep->i1 : 0;
+    p.epi_f0 = ep ? ep->f0 : 0.f;
+    p.epi_f1 = ep ? ep->f1 : 0.f;
     {
         static int dbg = -1;
         if (dbg < 0) {
@@ -1369,6 +1381,9 @@ extern "C" int llark_gemm_ex(const void* A, int a_mn_major, long long lda, const
         if (p.epi == LLARK_EPI_RELU_GLU && sel == 0 && !in_fp32)
             return two_cta ? launch2<0, 0, 0, 6>(ta, tb, p, max_ctas, stream)
                            : launch<0, 0, 0, 6>(ta, tb, p, max_ctas, stream);
+        if (p.epi == LLARK_EPI_CLAMP_GLU && sel == 0 && !in_fp32)
+            return two_cta ? launch2<0, 0, 0, 7>(ta, tb, p, max_ctas, stream)
+                           : launch<0, 0, 0, 7>(ta, tb, p, max_ctas, stream);
         return LLARK_EINVAL;
     }
     if (two_cta) {
@@ -1411,12 +1426,14 @@ extern "C" void llark_gemm_clear_cache(void) {
 // first row, rows <= 256, covering every run) and the CTA-pair kernel this is ONE launch whose m-blocks follow the list;
 // n_tiles is the list's length or, with seg_count_dev (a device word holding the real length), an upper bound of it, so
 // that nothing about the runs has to be known on the host. Without a tile list: seg_off_host [n_seg + 1] gives the run
-// boundaries and every run is a launch of its own. bf16 operands, bf16 or fp32 output. epi: LLARK_EPI_NONE or
-// LLARK_EPI_RELU2.
+// boundaries and every run is a launch of its own. bf16 operands, bf16 or fp32 output. epi: LLARK_EPI_NONE,
+// LLARK_EPI_RELU2 or LLARK_EPI_CLAMP_GLU (with f0, f1).
 extern "C" int llark_gemm_segments(const void* A, long long lda, const void* B, void* C, long long ldc, int c_fp32,
                                    const int* seg_off_host, int n_seg, const int* seg_tiles_dev, int n_tiles,
-                                   const int* seg_count_dev, int m_total, int N, int K, int epi, cudaStream_t stream) {
-    if (!A || !B || !C || n_seg <= 0 || N <= 0 || K <= 0 || (epi != LLARK_EPI_NONE && epi != LLARK_EPI_RELU2))
+                                   const int* seg_count_dev, int m_total, int N, int K, int epi, float f0, float f1,
+                                   cudaStream_t stream) {
+    if (!A || !B || !C || n_seg <= 0 || N <= 0 || K <= 0 || 
+        (epi != LLARK_EPI_NONE && epi != LLARK_EPI_RELU2 && epi != LLARK_EPI_CLAMP_GLU))
         return LLARK_EINVAL;
     if (seg_tiles_dev && n_tiles > 0 && llark_gemm_get_mode()) {
         if (m_total <= 0) return LLARK_EINVAL;
@@ -1427,6 +1444,8 @@ extern "C" int llark_gemm_segments(const void* A, long long lda, const void* B, 
         ep.ld = epi;
         ep.i0 = n_tiles;
         ep.i1 = n_seg;
+        ep.f0 = f0;
+        ep.f1 = f1;
         return llark_gemm_ex(A, 0, lda, B, 0, K, C, ldc, c_fp32, nullptr, 0, nullptr, 0, m_total, N, K, 0, 0, &ep, stream);
     }
     if (!seg_off_host) return LLARK_EINVAL;
@@ -1436,7 +1455,7 @@ extern "C" int llark_gemm_segments(const void* A, long long lda, const void* B, 
     for (int e = 0; e < n_seg; ++e) {
         const int r0 = seg_off_host[e], rows = seg_off_host[e + 1] - r0;
         if (rows <= 0) continue;
-        LlarkGemmEpilogue one = {epi, nullptr, nullptr, 0, 0, 0};
+        LlarkGemmEpilogue one = {epi, nullptr, nullptr, 0, 0, 0, f0, f1};
         const int rc = llark_gemm_ex(a + (long long)r0 * lda * 2, 0, lda, b + (long long)e * N * K * 2, 0, K,
                                      c + (long long)r0 * ldc * (c_fp32 ? 4 : 2), ldc, c_fp32, nullptr, 0, nullptr, 0, rows,
                                      N, K, 0, 0, &one, stream);

@@ -371,11 +371,12 @@ delta_scan_kernel(const float* __restrict__ vec, const float* __restrict__ v, lo
 }
 
 // ------------------------------------------------------------------------------------------------ read-out norm + gate
-// Warp per (token, head): y = o / sqrt(mean(o^2) + eps) * w * sigmoid(gate)   (gate_silu: * gate * sigmoid(gate))
+// Warp per (token, head): y = o / sqrt(mean(o^2) + eps) * w * sigmoid(gate)   (gate_silu: * gate * sigmoid(gate); w may be
+// missing). Row t of the output starts at out + t * out_ld.
 template <typename T>
 __global__ void head_norm_gate_kernel(const float* __restrict__ x, const float* __restrict__ w, int w_per_head,
                                       const float* __restrict__ gate, long long gate_ld, T* __restrict__ out,
-                                      long long n_items, int H, int E, float eps, int gate_silu) {
+                                      long long out_ld, long long n_items, int H, int E, float eps, int gate_silu) {
     const int lane = threadIdx.x & 31;
     const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     if (item >= n_items) return;
@@ -386,14 +387,73 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ x, const float* 
     for (int e = lane; e < E; e += 32) ss = fmaf(xr[e], xr[e], ss);
     ss = warp_sum(ss);
     const float r = 1.0f / sqrtf(ss / (float)E + eps);
-    const float* wr = w + (w_per_head ? (long long)h * E : 0);
+    const float* wr = w ? w + (w_per_head ? (long long)h * E : 0) : nullptr;
+    T* orow = out + t * out_ld + (long long)h * E;
     for (int e = lane; e < E; e += 32) {
-        float y = xr[e] * r * wr[e];
+        float y = xr[e] * r * (wr ? wr[e] : 1.0f);
         if (gate) {
             const float gv = gate[t * gate_ld + (long long)h * E + e];
             y *= gate_silu ? gv * sigmoidf_(gv) : sigmoidf_(gv);
         }
-        stf(out + item * E + e, y);
+        stf(orow + e, y);
+    }
+}
+
+// The same with 16-byte accesses and the head in registers from its one read to its write; a warp per head (several
+// heads per block), or BLOCK: a block per head, for norms over a whole projection).
+template <typename T, int NV, bool BLOCK>
+__global__ void head_norm_gate4_kernel(const float* __restrict__ x, const float* __restrict__ w, int w_per_head,
+                                       const float* __restrict__ gate, long long gate_ld, T* __restrict__ out,
+                                       long long out_ld, long long n_items, int H, int E, float eps, int gate_silu) {
+    __shared__ float red[32];
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+    const long long item = BLOCK ? (long long)blockIdx.x : (long long)blockIdx.x * nw + warp;
+    if (item >= n_items) return;  // (BLOCK: never)
+    const long long t = item / H;
+    const int h = (int)(item % H);
+    const int nv = E >> 2, first = BLOCK ? (int)threadIdx.x : lane, step = BLOCK ? (int)blockDim.x : 32;
+    const float4* xr = reinterpret_cast<const float4*>(x + item * E);
+    const float4* gr = gate ? reinterpret_cast<const float4*>(gate + t * gate_ld + (long long)h * E) : nullptr;
+    const float4* wr = w ? reinterpret_cast<const float4*>(w + (w_per_head ? (long long)h * E : 0)) : nullptr;
+    float4 v[NV], gv[NV];
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int c = first + i * step;
+        if (c < nv) {
+            v[i] = xr[c];
+            if (gr) gv[i] = gr[c];
+            ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+        }
+    }
+    ss = warp_sum(ss);
+    if (BLOCK) {
+        if (lane == 0) red[warp] = ss;
+        __syncthreads();
+        ss = 0.f;
+        for (int i = 0; i < nw; ++i) ss += red[i];
+    }
+    const float r = 1.0f / sqrtf(ss / (float)E + eps);
+    T* orow = out + t * out_ld + (long long)h * E;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int c = first + i * step;
+        if (c >= nv) continue;
+        float4 y = make_float4(v[i].x * r, v[i].y * r, v[i].z * r, v[i].w * r);
+        if (wr) {
+            const float4 ww = __ldg(wr + c);
+            y.x *= ww.x, y.y *= ww.y, y.z *= ww.z, y.w *= ww.w;
+        }
+        if (gr) {
+            const float4 g = gv[i];
+            y.x *= sigmoidf_(g.x), y.y *= sigmoidf_(g.y), y.z *= sigmoidf_(g.z), y.w *= sigmoidf_(g.w);
+            if (gate_silu) y.x *= g.x, y.y *= g.y, y.z *= g.z, y.w *= g.w;
+        }
+        if constexpr (sizeof(T) == 4) {
+            reinterpret_cast<float4*>(orow)[c] = y;
+        } else {
+            reinterpret_cast<uint2*>(orow)[c] = make_uint2(pack_bf16x2(y.x, y.y), pack_bf16x2(y.z, y.w));
+        }
     }
 }
 
@@ -596,17 +656,38 @@ extern "C" int llark_seq_delta_scan(const float* vec, const float* v, long long 
 }
 
 extern "C" int llark_seq_head_norm_gate(const float* x, const float* w, int w_per_head, const float* gate,
-                                        long long gate_ld, void* out, long long n_tok, int H, int E, float eps,
-                                        int gate_silu, int act_fp32, cudaStream_t st) {
-    if (n_tok <= 0 || H <= 0 || E <= 0 || !x || !w || !out) return LLARK_EINVAL;
+                                        long long gate_ld, void* out, long long out_ld, long long n_tok, int H, int E,
+                                        float eps, int gate_silu, int act_fp32, cudaStream_t st) {
+    if (n_tok <= 0 || H <= 0 || E <= 0 || !x || !out || out_ld < (long long)H * E) return LLARK_EINVAL;
     const long long items = n_tok * H;
+    auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+    const bool vec = E % 4 == 0 && al(x) && (!w || al(w)) && (!gate || (al(gate) && gate_ld % 4 == 0)) && al(out) && out_ld % 4 == 0;
+#define LLARK_HNG(T, NV, BLOCK, GRID, TH)                                                                               \
+    head_norm_gate4_kernel<T, NV, BLOCK><<<(unsigned)(GRID), TH, 0, st>>>(x, w, w_per_head, gate, gate_ld, (T*)out, out_ld, \
+                                                                         items, H, E, eps, gate_silu)
+#define LLARK_HNG_ALL(T)                                                                                                \
+    do {                                                                                                                \
+        if (E <= 128) LLARK_HNG(T, 1, false, (items + 3) / 4, 128);                                                     \
+        else if (E <= 256) LLARK_HNG(T, 2, false, (items + 3) / 4, 128);                                                \
+        else if (E <= 512) LLARK_HNG(T, 4, false, (items + 3) / 4, 128);                                                \
+        else if (E <= 2048) LLARK_HNG(T, 2, true, items, 256);                                                          \
+        else if (E <= 4096) LLARK_HNG(T, 2, true, items, 512);                                                          \
+        else LLARK_HNG(T, 4, true, items, 512);                                                                         \
+    } while (0)
+    if (vec && E <= 8192) {
+        if (act_fp32) LLARK_HNG_ALL(float);
+        else LLARK_HNG_ALL(__nv_bfloat16);
+        return check_launch();
+    }
+#undef LLARK_HNG_ALL
+#undef LLARK_HNG
     const unsigned grid = (unsigned)((items + 3) / 4);
     if (act_fp32)
-        head_norm_gate_kernel<float><<<grid, 128, 0, st>>>(x, w, w_per_head, gate, gate_ld, (float*)out, items, H, E, eps,
-                                                           gate_silu);
+        head_norm_gate_kernel<float><<<grid, 128, 0, st>>>(x, w, w_per_head, gate, gate_ld, (float*)out, out_ld, items, H, E,
+                                                           eps, gate_silu);
     else
         head_norm_gate_kernel<__nv_bfloat16><<<grid, 128, 0, st>>>(x, w, w_per_head, gate, gate_ld, (__nv_bfloat16*)out,
-                                                                   items, H, E, eps, gate_silu);
+                                                                   out_ld, items, H, E, eps, gate_silu);
     return check_launch();
 }
 

@@ -540,7 +540,7 @@ __global__ void swa_attn_kernel(const T* __restrict__ qn, const T* __restrict__ 
                                 const int* __restrict__ pos0, const int* __restrict__ slot, int H, int G, int D, int E,
                                 int window, int cap, int from_ring_only, const float* __restrict__ sink,
                                 int gate_per_head, int chunk, float softcap, const float* __restrict__ vfreq,
-                                int v_interleaved) {
+                                int v_interleaved, long long out_ld, float out_scale) {
     extern __shared__ float sm[];
     const int nw = blockDim.x >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     float* sq = sm;                      // [D]
@@ -679,9 +679,9 @@ __global__ void swa_attn_kernel(const T* __restrict__ qn, const T* __restrict__ 
             float o = 0.f;
             for (int w = 0; w < nw; ++w)
                 if (sm_m[w] != -INFINITY) o = fmaf(sacc[w * E + e], expf(sm_m[w] - mm), o);
-            o /= lt;
+            o = o / lt * out_scale;
             if (gate) o *= sigmoidf_(gate[(long long)t * gate_ld + (gate_per_head ? h : h * E + e)]);
-            stf(out + ((long long)t * H + h) * E + e, o);
+            stf(out + (long long)t * out_ld + h * E + e, o);
         }
         return;
     }
@@ -692,7 +692,7 @@ __global__ void swa_attn_kernel(const T* __restrict__ qn, const T* __restrict__ 
         float o = 0.f;
         for (int w = 0; w < nw; ++w)
             if (sm_m[w] != -INFINITY) o = fmaf(sacc[w * E + e], expf(sm_m[w] - mm), o);
-        so[e] = o / lt;
+        so[e] = o / lt * out_scale;
     }
     __syncthreads();
     const int half = E >> 1;
@@ -706,13 +706,13 @@ __global__ void swa_attn_kernel(const T* __restrict__ qn, const T* __restrict__ 
             a *= sigmoidf_(gate[(long long)t * gate_ld + (gate_per_head ? h : h * E + iu)]);
             bb *= sigmoidf_(gate[(long long)t * gate_ld + (gate_per_head ? h : h * E + iv)]);
         }
-        stf(out + ((long long)t * H + h) * E + iu, a);
-        stf(out + ((long long)t * H + h) * E + iv, bb);
+        stf(out + (long long)t * out_ld + h * E + iu, a);
+        stf(out + (long long)t * out_ld + h * E + iv, bb);
     }
     if ((E & 1) && threadIdx.x == 0) {  // an odd last channel has no partner and passes
         float o = so[E - 1];
         if (gate) o *= sigmoidf_(gate[(long long)t * gate_ld + (gate_per_head ? h : h * E + E - 1)]);
-        stf(out + ((long long)t * H + h) * E + E - 1, o);
+        stf(out + (long long)t * out_ld + h * E + E - 1, o);
     }
 }
 
@@ -1035,7 +1035,7 @@ static int launch_swa(const void* qn, const void* kn, const void* vv, const void
                       const float* gate, long long gate_ld, const float* scale_h, void* out, const int* tok_seq,
                       const int* cu, const int* pos0, const int* slot, int n_tok, int H, int G, int D, int E, int window,
                       int cap, int from_ring_only, const float* sink, int gate_per_head, int chunk, float softcap,
-                      const float* vfreq, int v_interleaved, cudaStream_t st) {
+                      const float* vfreq, int v_interleaved, long long out_ld, float out_scale, cudaStream_t st) {
     const int span = chunk > 0 ? chunk : window;  // most keys a query sees
     int nw = 1;
     while (nw < 8 && nw * 64 < span) nw <<= 1;  // two tiles per warp before another warp pays off
@@ -1046,7 +1046,7 @@ static int launch_swa(const void* qn, const void* kn, const void* vv, const void
     swa_attn_kernel<T, DPL><<<grid, nw * 32, smem, st>>>((const T*)qn, (const T*)kn, (const T*)vv, (const T*)kring, \
                                                          (const T*)vring, gate, gate_ld, scale_h, (T*)out, tok_seq, \
                                                          cu, pos0, slot, H, G, D, E, window, cap, from_ring_only, \
-                                                         sink, gate_per_head, chunk, softcap, vfreq, v_interleaved)
+                                                         sink, gate_per_head, chunk, softcap, vfreq, v_interleaved, out_ld, out_scale)
     if (dpl <= 1) LLARK_SWA(1);
     else if (dpl <= 2) LLARK_SWA(2);
     else if (dpl <= 4) LLARK_SWA(4);
@@ -1063,18 +1063,19 @@ extern "C" int llark_seq_swa_attn(const void* qn, const void* kn, const void* vv
                                   const int* tok_seq, const int* cu, const int* pos0, const int* slot, int n_tok, int H,
                                   int G, int D, int E, int window, int cap, int from_ring_only, const float* sink,
                                   int gate_per_head, int chunk, float softcap, const float* vfreq, int v_interleaved,
-                                  int act_fp32, cudaStream_t st) {
+                                  long long out_ld, float out_scale, int act_fp32, cudaStream_t st) {
     if (n_tok <= 0 || H <= 0 || G <= 0 || (H % G) || D <= 0 || E <= 0 || window <= 0 || cap <= 0 || !qn || !kring ||
-        !vring || !scale_h || !out || !tok_seq || !cu || !pos0 || !slot || chunk < 0 || softcap < 0.f)
+        !vring || !scale_h || !out || !tok_seq || !cu || !pos0 || !slot || chunk < 0 || softcap < 0.f ||
+        out_ld < (long long)H * E)
         return LLARK_EINVAL;
     if (!from_ring_only && (!kn || !vv)) return LLARK_EINVAL;
     if ((size_t)(D + 8 * 32 + 16 + 9 * E) * sizeof(float) > 48 * 1024) return LLARK_EINVAL;
     return act_fp32 ? launch_swa<float>(qn, kn, vv, kring, vring, gate, gate_ld, scale_h, out, tok_seq, cu, pos0, slot,
                                         n_tok, H, G, D, E, window, cap, from_ring_only, sink, gate_per_head, chunk,
-                                        softcap, vfreq, v_interleaved, st)
+                                        softcap, vfreq, v_interleaved, out_ld, out_scale, st)
                     : launch_swa<bf16_t>(qn, kn, vv, kring, vring, gate, gate_ld, scale_h, out, tok_seq, cu, pos0, slot,
                                          n_tok, H, G, D, E, window, cap, from_ring_only, sink, gate_per_head, chunk,
-                                         softcap, vfreq, v_interleaved, st);
+                                         softcap, vfreq, v_interleaved, out_ld, out_scale, st);
 }
 
 extern "C" int llark_seq_kv_ring_write(const void* kn, const void* vv, void* kring, void* vring, const int* tok_seq,

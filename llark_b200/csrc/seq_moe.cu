@@ -1,5 +1,5 @@
 // Routed mixture of experts on the generation path: every token uses `top` of n small feed-forwards
-// down(silu(gate x) * (up x)), or down(relu(up x)^2). The router picks experts on the device, one kernel sorts the (token, choice) entries by
+// down(silu(gate x) * (up x)), down(relu(up x)^2) or a clamped gated unit. The router picks experts on the device, one kernel sorts the (token, choice) entries by
 // expert and cuts each expert's run into row tiles, and two grouped GEMM launches walk that tile list (rows gathered
 // through the sort permutation). Large bf16 steps instead run every expert's rows through the tcgen05 GEMM core in its
 // rows-in-runs mode (llark_seq_moe_gather, llark_gemm_segments with the sort kernel's list of 256-row tiles and its
@@ -15,7 +15,8 @@
 //                           the best `keep` groups cannot be chosen; weights = the chosen experts' plain scores * scale,
 //                           not renormalised. Router outputs >= n_real are experts without weights that hand their input
 //                           through: the sort leaves them out of the tile lists, the residual kernel adds the input.
-//   llark_seq_moe_route_top   the `top` largest logits are chosen, weights = softmax over the chosen logits only
+//   llark_seq_moe_route_top   the `top` largest logits are chosen, weights = softmax over the chosen logits only, or their
+//                           sigmoids
 //   llark_seq_moe_sort      entries -> perm (sorted by expert), pos_of (inverse), tiles (expert, first row, rows)
 //   llark_seq_moe_up        act[pos] = silu(W_gate,e x) * (W_up,e x), or relu(W_up,e x)^2 for experts without a gate;
 //                           x = the entry's token row
@@ -209,9 +210,10 @@ __global__ void route_bias_kernel(const float* __restrict__ logits, long long ld
 }
 
 // Warp per token, logits in shared memory. The choice is made on the logits themselves (a softmax over all of them could
-// underflow and lose the order); ties go to the lower number.
+// underflow, a sigmoid saturate, and lose the order); ties go to the lower number. Weights: softmax over the chosen logits,
+// or, sigmoid_wts, the sigmoid of each as it is.
 __global__ void route_top_kernel(const float* __restrict__ logits, long long ld, int* __restrict__ ids,
-                                 float* __restrict__ wts, int n_tok, int n_exp, int top) {
+                                 float* __restrict__ wts, int n_tok, int n_exp, int top, int sigmoid_wts) {
     extern __shared__ float sm[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
     const long long t = (long long)blockIdx.x * nw + warp;
@@ -250,7 +252,7 @@ __global__ void route_top_kernel(const float* __restrict__ logits, long long ld,
     const float sum = warp_sum(w);
     if (lane < top) {
         ids[t * top + lane] = chosen_e;
-        wts[t * top + lane] = w / sum;
+        wts[t * top + lane] = sigmoid_wts ? sigmoidf_(chosen) : w / sum;
     }
 }
 
@@ -311,15 +313,29 @@ __global__ void sort_kernel(const int* __restrict__ ids, int n_ent, int n_exp, i
 // Block = one row tile of one expert x 64 output columns. MODE kSiluGlu: two weight matrices (gate rows, then up rows, of the
 // expert's [2 * N, K] block) and out = silu(a) * b; kRelu2: out = relu(product)^2; kPlain: the product. Rows of A:
 // gather ? perm[pos] / top : pos.
-enum { kPlain = 0, kSiluGlu = 1, kRelu2 = 2 };
+// kClampGlu: gate and up rows of the expert's [2 * N, K] block alternate, out = g' * sigmoid(slope g') * (u' + 1) with
+// g' = min(g, limit), u' = clamp(u, -limit, limit). in_wts (optional): entry i = perm[pos] of the step is multiplied by
+// in_wts[i] on its way in, which is done on the sums (W (c x) = c (W x)).
+enum { kPlain = 0, kSiluGlu = 1, kRelu2 = 2, kClampGlu = 3 };
+
+struct UpArgs {
+    const float* in_wts;
+    float limit, slope;
+};
+__device__ __forceinline__ float clamp_glu(const UpArgs& a, float g, float u) {
+    g = fminf(g, a.limit);
+    return g / (1.0f + expf(-a.slope * g)) * (fminf(fmaxf(u, -a.limit), a.limit) + 1.0f);
+}
 
 template <typename T, typename TC, int MODE>
 __global__ void __launch_bounds__(256)
 grouped_linear_kernel(const T* __restrict__ A, long long lda, const int* __restrict__ perm, int top,
                       const T* __restrict__ W, TC* __restrict__ Cm, long long ldc, const int* __restrict__ tiles,
-                      const int* __restrict__ meta, int N, int K) {
+                      const int* __restrict__ meta, int N, int K, UpArgs up) {
     constexpr int BM = kTileRows, BN = 64, BK = 16;
-    constexpr bool DUAL = MODE == kSiluGlu;
+    constexpr bool DUAL = MODE == kSiluGlu || MODE == kClampGlu;
+    constexpr int STEP = MODE == kClampGlu ? 2 : 1;  // weight rows from one gate (up) row to the next
+    const int up0 = MODE == kClampGlu ? 1 : N;       // the first up row
     if ((int)blockIdx.y >= meta[0]) return;
     __shared__ float As[BK][BM + 4];
     __shared__ float Ws[DUAL ? 2 : 1][BK][BN + 4];
@@ -336,8 +352,8 @@ grouped_linear_kernel(const T* __restrict__ A, long long lda, const int* __restr
             const int r = i / BK, k = i % BK;
             As[k][r] = (rows[r] >= 0 && k0 + k < K) ? ldf(A + (long long)rows[r] * lda + k0 + k) : 0.f;
             const bool in = n0 + r < N && k0 + k < K;
-            Ws[0][k][r] = in ? ldf(We + (long long)(n0 + r) * K + k0 + k) : 0.f;
-            if (DUAL) Ws[1][k][r] = in ? ldf(We + (long long)(N + n0 + r) * K + k0 + k) : 0.f;
+            Ws[0][k][r] = in ? ldf(We + (long long)(n0 + r) * STEP * K + k0 + k) : 0.f;
+            if (DUAL) Ws[1][k][r] = in ? ldf(We + ((long long)(n0 + r) * STEP + up0) * K + k0 + k) : 0.f;
         }
         __syncthreads();
 #pragma unroll
@@ -367,7 +383,10 @@ grouped_linear_kernel(const T* __restrict__ A, long long lda, const int* __restr
             const int m = ty * 4 + i, n = n0 + tx * 4 + j;
             if (m < nr && n < N) {
                 float y = acc[i][j];
-                if (DUAL) y = y * sigmoidf_(y) * acc2[i][j];
+                const float c = up.in_wts ? up.in_wts[perm[r0 + m]] : 1.0f;
+                y *= c;
+                if (MODE == kSiluGlu) y = y * sigmoidf_(y) * (c * acc2[i][j]);
+                if (MODE == kClampGlu) y = clamp_glu(up, y, c * acc2[i][j]);
                 if (MODE == kRelu2) {
                     y = fmaxf(y, 0.f);
                     y *= y;
@@ -377,7 +396,7 @@ grouped_linear_kernel(const T* __restrict__ A, long long lda, const int* __restr
         }
 }
 
-// Few rows per expert (decode): a warp owns one output column of one row tile (kSiluGlu: its gate and its up row) or two
+// Few rows per expert (decode): a warp owns one output column of one row tile (gated units: its gate and its up row) or two
 // adjacent ones (kPlain, kRelu2) and streams the two weight rows in 16-byte pieces; the tile's rows come from L1 / L2, MB at a
 // time, and are read once for both. A small MB keeps the registers few and the warps many, which pays as long as an expert
 // has a handful of rows (the second pass over a weight row comes from L1).
@@ -385,16 +404,17 @@ template <typename T, typename TC, int MODE, int MB>
 __global__ void __launch_bounds__(256)
 grouped_rows_kernel(const T* __restrict__ A, long long lda, const int* __restrict__ perm, int top,
                     const T* __restrict__ W, TC* __restrict__ Cm, long long ldc, const int* __restrict__ tiles,
-                    const int* __restrict__ meta, int N, int K, int vec_ok) {
+                    const int* __restrict__ meta, int N, int K, int vec_ok, UpArgs up) {
     constexpr int VEC = 16 / (int)sizeof(T);
-    constexpr bool DUAL = MODE == kSiluGlu;
+    constexpr bool DUAL = MODE == kSiluGlu || MODE == kClampGlu;
     if ((int)blockIdx.y >= meta[0]) return;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int n = (blockIdx.x * (blockDim.x >> 5) + warp) * (DUAL ? 1 : 2);
     if (n >= N) return;
     const int ex = tiles[3 * blockIdx.y], r0 = tiles[3 * blockIdx.y + 1], nr = tiles[3 * blockIdx.y + 2];
-    const T* w1 = W + ((long long)ex * (DUAL ? 2 : 1) * N + n) * K;
-    const T* w2 = w1 + (DUAL ? (long long)N * K : (n + 1 < N ? (long long)K : 0));  // tail: re-read, never stored
+    const T* w1 = W + ((long long)ex * (DUAL ? 2 : 1) * N + (MODE == kClampGlu ? 2 * n : n)) * K;
+    const T* w2 = w1 + (MODE == kSiluGlu ? (long long)N * K
+                                         : (MODE == kClampGlu || n + 1 < N ? (long long)K : 0));  // tail: re-read, never stored
     for (int m0 = 0; m0 < nr; m0 += MB) {
         const T* ar[MB];
 #pragma unroll
@@ -442,7 +462,12 @@ grouped_rows_kernel(const T* __restrict__ A, long long lda, const int* __restric
 #pragma unroll
         for (int m = 0; m < MB; ++m) {
             float y = warp_sum(acc[m]), u = warp_sum(acc2[m]);
-            if (DUAL) y = y * sigmoidf_(y) * u;
+            if (up.in_wts && m0 + m < nr) {
+                const float c = up.in_wts[perm[r0 + m0 + m]];
+                y *= c, u *= c;
+            }
+            if (MODE == kSiluGlu) y = y * sigmoidf_(y) * u;
+            if (MODE == kClampGlu) y = clamp_glu(up, y, u);
             if (MODE == kRelu2) {
                 y = fmaxf(y, 0.f), u = fmaxf(u, 0.f);
                 y *= y, u *= u;
@@ -457,20 +482,29 @@ grouped_rows_kernel(const T* __restrict__ A, long long lda, const int* __restric
 }
 
 // ------------------------------------------------------------------------------------------------ dense-GEMM route
-// Large steps run each expert's rows through the framework's GEMM core instead: rows gathered into sorted order first,
-// silu(gate) * up afterwards.
+// Large steps run each expert's rows through the framework's GEMM core instead: rows gathered into sorted order first (each
+// multiplied by its weight where the unit wants it so), silu(gate) * up afterwards.
 template <typename T>
 __global__ void gather_rows_kernel(const T* __restrict__ x, long long ldx, const int* __restrict__ perm, int top,
-                                   T* __restrict__ xs, int C) {
+                                   T* __restrict__ xs, int C, const float* __restrict__ in_wts) {
     const long long p = blockIdx.x;
     const T* src = x + (long long)(perm[p] / top) * ldx;
     T* dst = xs + p * C;
+    const float c = in_wts ? in_wts[perm[p]] : 1.0f;
     if ((C * (int)sizeof(T)) % 16 == 0 && (ldx * (long long)sizeof(T)) % 16 == 0) {
-        const int nv = C * (int)sizeof(T) / 16;
-        for (int i = threadIdx.x; i < nv; i += blockDim.x)
-            reinterpret_cast<uint4*>(dst)[i] = reinterpret_cast<const uint4*>(src)[i];
+        constexpr int VEC = 16 / (int)sizeof(T);
+        const int nv = C / VEC;
+        for (int i = threadIdx.x; i < nv; i += blockDim.x) {
+            uint4 v = reinterpret_cast<const uint4*>(src)[i];
+            if (in_wts) {
+                T* e = reinterpret_cast<T*>(&v);
+#pragma unroll
+                for (int j = 0; j < VEC; ++j) stf(e + j, c * ldf(e + j));
+            }
+            reinterpret_cast<uint4*>(dst)[i] = v;
+        }
     } else {
-        for (int i = threadIdx.x; i < C; i += blockDim.x) dst[i] = src[i];
+        for (int i = threadIdx.x; i < C; i += blockDim.x) stf(dst + i, c * ldf(src + i));
     }
 }
 
@@ -520,12 +554,12 @@ extern "C" int llark_seq_moe_route_bias(const float* logits, long long ld, const
 }
 
 extern "C" int llark_seq_moe_route_top(const float* logits, long long ld, int* ids, float* wts, int n_tok, int n_exp, int top,
-                                       cudaStream_t st) {
+                                       int sigmoid_wts, cudaStream_t st) {
     if (n_tok <= 0 || n_exp <= 0 || top <= 0 || top > 32 || top > n_exp || !logits || !ids || !wts) return LLARK_EINVAL;
     const int nw = 4;
     const size_t smem = sizeof(float) * nw * (size_t)n_exp;
     if (smem > 48 * 1024) return LLARK_EINVAL;
-    route_top_kernel<<<(n_tok + nw - 1) / nw, nw * 32, smem, st>>>(logits, ld, ids, wts, n_tok, n_exp, top);
+    route_top_kernel<<<(n_tok + nw - 1) / nw, nw * 32, smem, st>>>(logits, ld, ids, wts, n_tok, n_exp, top, sigmoid_wts);
     return check_launch();
 }
 
@@ -543,44 +577,45 @@ extern "C" int llark_seq_moe_sort(const int* ids, int n_ent, int n_exp, int n_re
 
 template <typename T, typename TC, int MODE>
 static void launch_rows(const T* A, long long lda, const int* perm, int top, const T* W, TC* C, const int* tiles,
-                        const int* meta, int max_tiles, int n_ent, int N, int K, int vec_ok, cudaStream_t st) {
-    const int per = MODE == kSiluGlu ? 8 : 16;  // output columns of a block's eight warps
+                        const int* meta, int max_tiles, int n_ent, int N, int K, int vec_ok, UpArgs up, cudaStream_t st) {
+    const int per = MODE == kSiluGlu || MODE == kClampGlu ? 8 : 16;  // output columns of a block's eight warps
     const dim3 grid((N + per - 1) / per, max_tiles);
     const int n_exp = max_tiles - (n_ent + kTileRows - 1) / kTileRows;
     if (n_ent <= 8 * n_exp)  // a handful of rows per expert
-        grouped_rows_kernel<T, TC, MODE, 2><<<grid, 256, 0, st>>>(A, lda, perm, top, W, C, N, tiles, meta, N, K, vec_ok);
+        grouped_rows_kernel<T, TC, MODE, 2><<<grid, 256, 0, st>>>(A, lda, perm, top, W, C, N, tiles, meta, N, K, vec_ok, up);
     else
-        grouped_rows_kernel<T, TC, MODE, 8><<<grid, 256, 0, st>>>(A, lda, perm, top, W, C, N, tiles, meta, N, K, vec_ok);
+        grouped_rows_kernel<T, TC, MODE, 8><<<grid, 256, 0, st>>>(A, lda, perm, top, W, C, N, tiles, meta, N, K, vec_ok, up);
 }
 
 template <typename T, int MODE>
 static int launch_up(const void* x, long long ldx, const int* perm, int top, const void* w, void* act, const int* tiles,
-                     const int* meta, int max_tiles, int n_ent, int ff, int K, cudaStream_t st) {
+                     const int* meta, int max_tiles, int n_ent, int ff, int K, UpArgs up, cudaStream_t st) {
     if (n_ent <= kRowsRouteMaxEntries) {  // a handful of rows per expert: stream the weights once
         const int vec = 16 / (int)sizeof(T);
         const int vec_ok = (K % vec == 0) && (ldx % vec == 0) &&
                            (((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w)) & 15) == 0);
         launch_rows<T, T, MODE>((const T*)x, ldx, perm, top, (const T*)w, (T*)act, tiles, meta, max_tiles, n_ent, ff, K,
-                                vec_ok, st);
+                                vec_ok, up, st);
     } else {
         grouped_linear_kernel<T, T, MODE><<<dim3((ff + 63) / 64, max_tiles), 256, 0, st>>>(
-            (const T*)x, ldx, perm, top, (const T*)w, (T*)act, ff, tiles, meta, ff, K);
+            (const T*)x, ldx, perm, top, (const T*)w, (T*)act, ff, tiles, meta, ff, K, up);
     }
     return check_launch();
 }
 
 // gated = 1: w holds gate rows, then up rows, [n, 2 * ff, K], act = silu(gate x) * (up x); gated = 0: w is [n, ff, K],
-// act = relu(w x)^2
+// act = relu(w x)^2; gated = 2: gate and up rows alternate, the clamped gated unit with `limit` and `slope`
 extern "C" int llark_seq_moe_up(const void* x, long long ldx, const int* perm, int top, const void* w, void* act,
                                 const int* tiles, const int* meta, int max_tiles, int n_ent, int ff, int K, int gated,
-                                int act_fp32, cudaStream_t st) {
-    if (max_tiles <= 0 || ff <= 0 || K <= 0 || top <= 0 || !x || !perm || !w || !act || !tiles || !meta)
+                                const float* in_wts, float limit, float slope, int act_fp32, cudaStream_t st) {
+    if (max_tiles <= 0 || ff <= 0 || K <= 0 || top <= 0 || gated < 0 || gated > 2 || !x || !perm || !w || !act || !tiles || !meta)
         return LLARK_EINVAL;
-    if (gated)
-        return act_fp32 ? launch_up<float, kSiluGlu>(x, ldx, perm, top, w, act, tiles, meta, max_tiles, n_ent, ff, K, st)
-                        : launch_up<bf16_t, kSiluGlu>(x, ldx, perm, top, w, act, tiles, meta, max_tiles, n_ent, ff, K, st);
-    return act_fp32 ? launch_up<float, kRelu2>(x, ldx, perm, top, w, act, tiles, meta, max_tiles, n_ent, ff, K, st)
-                    : launch_up<bf16_t, kRelu2>(x, ldx, perm, top, w, act, tiles, meta, max_tiles, n_ent, ff, K, st);
+    const UpArgs up{in_wts, limit, slope};
+#define LLARK_UP(T, MODE) launch_up<T, MODE>(x, ldx, perm, top, w, act, tiles, meta, max_tiles, n_ent, ff, K, up, st)
+    if (gated == 2) return act_fp32 ? LLARK_UP(float, kClampGlu) : LLARK_UP(bf16_t, kClampGlu);
+    if (gated == 1) return act_fp32 ? LLARK_UP(float, kSiluGlu) : LLARK_UP(bf16_t, kSiluGlu);
+    return act_fp32 ? LLARK_UP(float, kRelu2) : LLARK_UP(bf16_t, kRelu2);
+#undef LLARK_UP
 }
 
 extern "C" int llark_seq_moe_down(const void* act, const void* w_down, float* z, const int* tiles, const int* meta,
@@ -592,29 +627,29 @@ extern "C" int llark_seq_moe_down(const void* act, const void* w_down, float* z,
                            (((reinterpret_cast<uintptr_t>(act) | reinterpret_cast<uintptr_t>(w_down)) & 15) == 0);
         if (act_fp32)
             launch_rows<float, float, kPlain>((const float*)act, ff, nullptr, 1, (const float*)w_down, z, tiles, meta,
-                                              max_tiles, n_ent, C, ff, vec_ok, st);
+                                              max_tiles, n_ent, C, ff, vec_ok, UpArgs{}, st);
         else
             launch_rows<bf16_t, float, kPlain>((const bf16_t*)act, ff, nullptr, 1, (const bf16_t*)w_down, z, tiles, meta,
-                                               max_tiles, n_ent, C, ff, vec_ok, st);
+                                               max_tiles, n_ent, C, ff, vec_ok, UpArgs{}, st);
         return check_launch();
     }
     dim3 grid((C + 63) / 64, max_tiles);
     if (act_fp32)
         grouped_linear_kernel<float, float, kPlain><<<grid, 256, 0, st>>>((const float*)act, ff, nullptr, 1,
-                                                                         (const float*)w_down, z, C, tiles, meta, C, ff);
+                                                                         (const float*)w_down, z, C, tiles, meta, C, ff, UpArgs{});
     else
         grouped_linear_kernel<bf16_t, float, kPlain><<<grid, 256, 0, st>>>((const bf16_t*)act, ff, nullptr, 1,
-                                                                          (const bf16_t*)w_down, z, C, tiles, meta, C, ff);
+                                                                          (const bf16_t*)w_down, z, C, tiles, meta, C, ff, UpArgs{});
     return check_launch();
 }
 
 extern "C" int llark_seq_moe_gather(const void* x, long long ldx, const int* perm, int top, void* xs, int n_ent, int C,
-                                    int act_fp32, cudaStream_t st) {
+                                    const float* in_wts, int act_fp32, cudaStream_t st) {
     if (n_ent <= 0 || C <= 0 || top <= 0 || !x || !perm || !xs) return LLARK_EINVAL;
     if (act_fp32)
-        gather_rows_kernel<float><<<n_ent, 128, 0, st>>>((const float*)x, ldx, perm, top, (float*)xs, C);
+        gather_rows_kernel<float><<<n_ent, 128, 0, st>>>((const float*)x, ldx, perm, top, (float*)xs, C, in_wts);
     else
-        gather_rows_kernel<bf16_t><<<n_ent, 128, 0, st>>>((const bf16_t*)x, ldx, perm, top, (bf16_t*)xs, C);
+        gather_rows_kernel<bf16_t><<<n_ent, 128, 0, st>>>((const bf16_t*)x, ldx, perm, top, (bf16_t*)xs, C, in_wts);
     return check_launch();
 }
 

@@ -62,7 +62,7 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
 template <typename T>
 __global__ void embed_kernel(const int* __restrict__ ids, const int* __restrict__ tok_seq, const int* __restrict__ cu,
                              const int* __restrict__ pos0, const T* __restrict__ table, const T* __restrict__ pos_table,
-                             float scale, float* __restrict__ x, int C) {
+                             float scale, float* __restrict__ x, T* __restrict__ x_act, int C) {
     const int t = blockIdx.x;
     const int b = tok_seq[t];
     const long long p = pos0[b] + (t - cu[b]);
@@ -72,6 +72,7 @@ __global__ void embed_kernel(const int* __restrict__ ids, const int* __restrict_
         float v = ldf(e + c) * scale;
         if (pe) v += ldf(pe + c);
         x[(long long)t * C + c] = v;
+        if (x_act) stf(x_act + (long long)t * C + c, v);
     }
 }
 
@@ -396,6 +397,160 @@ __global__ void gated_norm_add_kernel(const float* __restrict__ x, const float* 
     for (int c = threadIdx.x; c < C; c += blockDim.x) stf(xa + c, rowbuf[c] * r2 * w_next[c]);  // each thread reads its own
 }
 
+// ------------------------------------------------------------------------------------------------ layer norm
+// Layer norm (mean off, divided by the root of the mean squared deviation + eps, times a weight, no offset) around a residual
+// sum, one row per block:
+//     f = y (optional) + the rows pos_of[t * top + k] of z, k = 0 .. top - 1 in order (times wts[t, k] when given)
+//     o = x + norm(f) * w_post    (w_post NULL: x + f)           -> x_out (optional)
+//     norm(o) * w_next            (w_next NULL: o itself)        -> x_act (optional)
+// x = row rows[t] of x when rows is given; without y and z there is no f: the plain norm of x.
+struct LnArgs {
+    const float* x;
+    const int* rows;
+    const float *y, *z;
+    const int* pos_of;
+    const float* wts;
+    int top;
+    const float *w_post, *w_next;
+    float* x_out;
+    int C;
+    float eps;
+};
+__device__ __forceinline__ float4 add4(float4 a, float4 b) { return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w); }
+__device__ __forceinline__ float4 sub1(float4 a, float m) { return make_float4(a.x - m, a.y - m, a.z - m, a.w - m); }
+__device__ __forceinline__ float dot4(float4 a) { return a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w; }
+__device__ __forceinline__ float4 scale4(float4 a, float r, float4 w) {
+    return make_float4(a.x * r * w.x, a.y * r * w.y, a.z * r * w.z, a.w * r * w.w);
+}
+
+// C % 4 == 0, 16-byte pointers, C <= 4 * NV * blockDim.x: the row stays in registers from its first read to its last write.
+template <typename T, int NV>
+__global__ void layer_norm_add4_kernel(LnArgs p, T* __restrict__ x_act) {
+    __shared__ float red[32];
+    const long long t = blockIdx.x, src = p.rows ? p.rows[t] : t;
+    const int nv = p.C >> 2;
+    const float4* xr = reinterpret_cast<const float4*>(p.x + src * p.C);
+    float4 o[NV];
+    if (p.y || p.z) {
+        float4 f[NV];
+        float s = 0.f;
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const int v = threadIdx.x + i * blockDim.x;
+            f[i] = o[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (v < nv) {
+                o[i] = xr[v];
+                if (p.y) f[i] = reinterpret_cast<const float4*>(p.y + t * p.C)[v];
+#pragma unroll 4
+                for (int k = 0; k < p.top; ++k) {
+                    const float4 e = __ldg(reinterpret_cast<const float4*>(p.z + (long long)__ldg(p.pos_of + t * p.top + k) * p.C) + v);
+                    const float wt = p.wts ? __ldg(p.wts + t * p.top + k) : 1.0f;
+                    f[i] = make_float4(fmaf(wt, e.x, f[i].x), fmaf(wt, e.y, f[i].y), fmaf(wt, e.z, f[i].z), fmaf(wt, e.w, f[i].w));
+                }
+                s += (f[i].x + f[i].y) + (f[i].z + f[i].w);
+            }
+        }
+        if (p.w_post) {
+            const float mean = block_sum(s, red) / (float)p.C;
+            float ss = 0.f;
+#pragma unroll
+            for (int i = 0; i < NV; ++i)
+                if (threadIdx.x + i * blockDim.x < nv) {
+                    f[i] = sub1(f[i], mean);
+                    ss += dot4(f[i]);
+                }
+            const float r = 1.0f / sqrtf(block_sum(ss, red) / (float)p.C + p.eps);
+#pragma unroll
+            for (int i = 0; i < NV; ++i) {
+                const int v = threadIdx.x + i * blockDim.x;
+                if (v < nv) f[i] = scale4(f[i], r, __ldg(reinterpret_cast<const float4*>(p.w_post) + v));
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < NV; ++i) o[i] = add4(o[i], f[i]);
+    } else {
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const int v = threadIdx.x + i * blockDim.x;
+            o[i] = v < nv ? xr[v] : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+    }
+    if (p.x_out) {
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const int v = threadIdx.x + i * blockDim.x;
+            if (v < nv) reinterpret_cast<float4*>(p.x_out + t * p.C)[v] = o[i];
+        }
+    }
+    if (!x_act) return;
+    float r = 1.0f;
+    if (p.w_next) {
+        float s = 0.f, ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < NV; ++i) s += (o[i].x + o[i].y) + (o[i].z + o[i].w);  // zeros behind the row's end
+        const float mean = block_sum(s, red) / (float)p.C;
+#pragma unroll
+        for (int i = 0; i < NV; ++i)
+            if (threadIdx.x + i * blockDim.x < nv) {
+                o[i] = sub1(o[i], mean);
+                ss += dot4(o[i]);
+            }
+        r = 1.0f / sqrtf(block_sum(ss, red) / (float)p.C + p.eps);
+    }
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int v = threadIdx.x + i * blockDim.x;
+        if (v < nv) {
+            const float4 h = p.w_next ? scale4(o[i], r, __ldg(reinterpret_cast<const float4*>(p.w_next) + v)) : o[i];
+            st4(x_act + t * p.C + 4 * v, h.x, h.y, h.z, h.w);
+        }
+    }
+}
+
+// Any C: the row in shared memory.
+template <typename T>
+__global__ void layer_norm_add_kernel(LnArgs p, T* __restrict__ x_act) {
+    extern __shared__ __align__(16) float rowbuf[];
+    __shared__ float red[32];
+    const long long t = blockIdx.x, src = p.rows ? p.rows[t] : t;
+    const int C = p.C;
+    const float* xr = p.x + src * C;
+    if (p.y || p.z) {
+        float s = 0.f;
+        for (int c = threadIdx.x; c < C; c += blockDim.x) {
+            float f = p.y ? p.y[t * C + c] : 0.f;
+            for (int k = 0; k < p.top; ++k)
+                f = fmaf(p.wts ? p.wts[t * p.top + k] : 1.0f, p.z[(long long)p.pos_of[t * p.top + k] * C + c], f);
+            rowbuf[c] = f;  // every thread keeps to its own entries
+            s += f;
+        }
+        float mean = 0.f, r = 1.f;
+        if (p.w_post) {
+            mean = block_sum(s, red) / (float)C;
+            float ss = 0.f;
+            for (int c = threadIdx.x; c < C; c += blockDim.x) ss = fmaf(rowbuf[c] - mean, rowbuf[c] - mean, ss);
+            r = 1.0f / sqrtf(block_sum(ss, red) / (float)C + p.eps);
+        }
+        for (int c = threadIdx.x; c < C; c += blockDim.x)
+            rowbuf[c] = xr[c] + (p.w_post ? (rowbuf[c] - mean) * r * p.w_post[c] : rowbuf[c]);
+    } else {
+        for (int c = threadIdx.x; c < C; c += blockDim.x) rowbuf[c] = xr[c];
+    }
+    if (p.x_out)
+        for (int c = threadIdx.x; c < C; c += blockDim.x) p.x_out[t * C + c] = rowbuf[c];
+    if (!x_act) return;
+    float mean = 0.f, r = 1.f;
+    if (p.w_next) {
+        float s = 0.f, ss = 0.f;
+        for (int c = threadIdx.x; c < C; c += blockDim.x) s += rowbuf[c];
+        mean = block_sum(s, red) / (float)C;
+        for (int c = threadIdx.x; c < C; c += blockDim.x) ss = fmaf(rowbuf[c] - mean, rowbuf[c] - mean, ss);
+        r = 1.0f / sqrtf(block_sum(ss, red) / (float)C + p.eps);
+    }
+    for (int c = threadIdx.x; c < C; c += blockDim.x)
+        stf(x_act + t * C + c, p.w_next ? (rowbuf[c] - mean) * r * p.w_next[c] : rowbuf[c]);
+}
+
 // ------------------------------------------------------------------------------------------------ tanh norm
 // tanh(alpha * v) * w + b: no mean, no variance, so a row needs no reduction and its columns spread over blocks (grid: rows
 // x column blocks). tanhf: the squashing belongs to what is computed in full fp32.
@@ -485,12 +640,24 @@ __global__ void tanh_kernel(const float* __restrict__ u, T* __restrict__ y, long
 }
 
 // ------------------------------------------------------------------------------------------------ linears
+// Activation of a product. The paired kinds take two adjacent columns, a gate and its up column, to one result.
+struct ActArg {
+    int kind;
+    float limit, slope;  // LLARK_ACT_CLAMP_GLU
+};
+__host__ __device__ __forceinline__ bool paired(int kind) { return kind == LLARK_ACT_RELU_GLU || kind == LLARK_ACT_CLAMP_GLU; }
+__device__ __forceinline__ float glu(const ActArg& a, float g, float u) {
+    if (a.kind == LLARK_ACT_RELU_GLU) return fmaxf(g, 0.f) * u;
+    g = fminf(g, a.limit);
+    return g / (1.0f + expf(-a.slope * g)) * (fminf(fmaxf(u, -a.limit), a.limit) + 1.0f);
+}
+
 // Few rows (decode): a warp owns NC adjacent output columns, its lanes stride over K in 16-byte pieces (streamed,
 // evict-first), the rows of A come from L1 / L2 and are read once per NC weight pieces.
 template <typename T, typename TC, int MB, int NC>
 __global__ void __launch_bounds__(256)
 linear_rows_kernel(const T* __restrict__ A, long long lda, const T* __restrict__ W, long long ldw, TC* __restrict__ Cm,
-                   long long ldc, const float* __restrict__ bias, int M, int N, int K, int vec_ok, int act) {
+                   long long ldc, const float* __restrict__ bias, int M, int N, int K, int vec_ok, ActArg act) {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const long long n0 = ((long long)blockIdx.x * (blockDim.x >> 5) + warp) * NC;
     const int m0 = blockIdx.y * MB;
@@ -536,12 +703,12 @@ linear_rows_kernel(const T* __restrict__ A, long long lda, const T* __restrict__
                 if (m0 + m < M) acc[m][c] = fmaf(ldf(A + (long long)(m0 + m) * lda + k), wv, acc[m][c]);
         }
     }
-    if (NC == 2 && act == LLARK_ACT_RELU_GLU) {  // the warp's two columns are a gate and its up column (N is even)
+    if (NC == 2 && paired(act.kind)) {  // the warp's two columns are a gate and its up column (N is even)
 #pragma unroll
         for (int m = 0; m < MB; ++m) {
             const float g = warp_sum(acc[m][0]) + (bias ? bias[n0] : 0.f);
             const float u = warp_sum(acc[m][NC - 1]) + (bias ? bias[n0 + 1] : 0.f);
-            if (lane == 0 && m0 + m < M) stf(Cm + (long long)(m0 + m) * ldc + (n0 >> 1), fmaxf(g, 0.f) * u);
+            if (lane == 0 && m0 + m < M) stf(Cm + (long long)(m0 + m) * ldc + (n0 >> 1), glu(act, g, u));
         }
         return;
     }
@@ -552,7 +719,7 @@ linear_rows_kernel(const T* __restrict__ A, long long lda, const T* __restrict__
             float s = warp_sum(acc[m][c]);
             if (lane == 0 && m0 + m < M && n0 + c < N) {
                 s += bias ? bias[n0 + c] : 0.f;
-                if (act == LLARK_ACT_RELU2) {
+                if (act.kind == LLARK_ACT_RELU2) {
                     s = fmaxf(s, 0.f);
                     s *= s;
                 }
@@ -565,7 +732,7 @@ linear_rows_kernel(const T* __restrict__ A, long long lda, const T* __restrict__
 template <typename T, typename TC, typename TW = T>
 __global__ void __launch_bounds__(256)
 linear_simt_kernel(const T* __restrict__ A, long long lda, const TW* __restrict__ W, long long ldw, TC* __restrict__ Cm,
-                   long long ldc, const float* __restrict__ bias, int M, int N, int K, int act) {
+                   long long ldc, const float* __restrict__ bias, int M, int N, int K, ActArg act) {
     constexpr int BM = 64, BN = 64, BK = 16;
     __shared__ float As[BK][BM + 4];
     __shared__ float Ws[BK][BN + 4];
@@ -600,13 +767,13 @@ linear_simt_kernel(const T* __restrict__ A, long long lda, const TW* __restrict_
             const int m = m0 + ty * 4 + i, n = n0 + tx * 4 + j;
             if (m >= M || n >= N) continue;
             float s = acc[i][j] + (bias ? bias[n] : 0.f);
-            if (act == LLARK_ACT_RELU_GLU) {  // n even: the gate; its up column is the next one of this thread (N is even)
+            if (paired(act.kind)) {  // n even: the gate; its up column is the next one of this thread (N is even)
                 if (j & 1) continue;
                 const float u = acc[i][(j + 1) & 3] + (bias ? bias[n + 1] : 0.f);
-                stf(Cm + (long long)m * ldc + (n >> 1), fmaxf(s, 0.f) * u);
+                stf(Cm + (long long)m * ldc + (n >> 1), glu(act, s, u));
                 continue;
             }
-            if (act == LLARK_ACT_RELU2) {
+            if (act.kind == LLARK_ACT_RELU2) {
                 s = fmaxf(s, 0.f);
                 s *= s;
             }
@@ -887,9 +1054,9 @@ __global__ void linear_rows_w32_kernel(const TA* __restrict__ A, long long lda, 
 }
 
 static bool bad_act(int act, int N) {
-    return act < LLARK_ACT_NONE || act > LLARK_ACT_RELU_GLU || (act == LLARK_ACT_RELU_GLU && (N % 2));
+    return act < LLARK_ACT_NONE || act > LLARK_ACT_CLAMP_GLU || (paired(act) && (N % 2));
 }
-static long long out_cols(int act, int N) { return act == LLARK_ACT_RELU_GLU ? N / 2 : N; }
+static long long out_cols(int act, int N) { return paired(act) ? N / 2 : N; }
 
 static int norm_threads(int C) {
     int t = 32;
@@ -905,16 +1072,16 @@ using namespace llark::seq;
 typedef __nv_bfloat16 bf16_t;
 
 extern "C" int llark_seq_embed(const int* ids, const int* tok_seq, const int* cu, const int* pos0, const void* table,
-                               const void* pos_table, float scale, float* x, int n_tok, int C, int act_fp32,
-                               cudaStream_t st) {
+                               const void* pos_table, float scale, float* x, void* x_act, int n_tok, int C,
+                               int act_fp32, cudaStream_t st) {
     if (n_tok <= 0 || C <= 0 || !ids || !tok_seq || !cu || !pos0 || !table || !x) return LLARK_EINVAL;
     const int th = norm_threads(C);
     if (act_fp32)
         embed_kernel<float><<<n_tok, th, 0, st>>>(ids, tok_seq, cu, pos0, (const float*)table, (const float*)pos_table,
-                                                  scale, x, C);
+                                                  scale, x, (float*)x_act, C);
     else
         embed_kernel<bf16_t><<<n_tok, th, 0, st>>>(ids, tok_seq, cu, pos0, (const bf16_t*)table,
-                                                   (const bf16_t*)pos_table, scale, x, C);
+                                                   (const bf16_t*)pos_table, scale, x, (bf16_t*)x_act, C);
     return check_launch();
 }
 
@@ -1081,6 +1248,51 @@ extern "C" int llark_seq_tanh_norm_add(const float* x, const float* y, const flo
     return check_launch();
 }
 
+extern "C" int llark_seq_layer_norm_add(const float* x, const int* rows, const float* y, const float* z, const int* pos_of,
+                                        const float* wts, int top, const float* w_post, const float* w_next, float* x_out,
+                                        void* x_act, long long n_rows, int C, float eps, int act_fp32, cudaStream_t st) {
+    if (n_rows <= 0 || C <= 0 || top < 0 || !x || (!x_out && !x_act) || (top > 0) != (z != nullptr) || (z && !pos_of) ||
+        (rows && (y || z || x_out)))
+        return LLARK_EINVAL;
+    const LnArgs p{x, rows, y, z, pos_of, wts, top, w_post, w_next, x_out, C, eps};
+    if (C % 4 == 0 && C <= 4 * 4 * 512 && aligned16({x, y, z, w_post, w_next, x_out, x_act})) {
+        const int nv = C / 4;
+        const int per = nv <= 256 ? 1 : (nv <= 1024 ? 2 : 4);  // float4 per thread
+        const int threads = ((nv + per - 1) / per + 31) / 32 * 32;
+#define LLARK_LN4(T, NV) layer_norm_add4_kernel<T, NV><<<(unsigned)n_rows, threads, 0, st>>>(p, (T*)x_act)
+        if (act_fp32) {
+            if (per == 1) LLARK_LN4(float, 1);
+            else if (per == 2) LLARK_LN4(float, 2);
+            else LLARK_LN4(float, 4);
+        } else {
+            if (per == 1) LLARK_LN4(bf16_t, 1);
+            else if (per == 2) LLARK_LN4(bf16_t, 2);
+            else LLARK_LN4(bf16_t, 4);
+        }
+#undef LLARK_LN4
+        return check_launch();
+    }
+    const size_t smem = sizeof(float) * (size_t)C;
+    if (smem > 200 * 1024) return LLARK_EINVAL;
+    const int threads = C < 64 ? 64 : (C > 512 ? 512 : (C + 31) / 32 * 32);
+#define LLARK_LN(T)                                                                                                   \
+    do {                                                                                                              \
+        if (smem > 48 * 1024) {                                                                                       \
+            cudaError_t e = cudaFuncSetAttribute(layer_norm_add_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
+                                                 (int)smem);                                                          \
+            if (e != cudaSuccess) {                                                                                   \
+                g_last_cuda_error = (int)e;                                                                           \
+                return LLARK_ECUDA;                                                                                   \
+            }                                                                                                         \
+        }                                                                                                             \
+        layer_norm_add_kernel<T><<<(unsigned)n_rows, threads, smem, st>>>(p, (T*)x_act);                              \
+    } while (0)
+    if (act_fp32) LLARK_LN(float);
+    else LLARK_LN(bf16_t);
+#undef LLARK_LN
+    return check_launch();
+}
+
 extern "C" int llark_seq_rmsnorm_rows(const float* x, const int* rows, const float* w, void* out, int n_rows, int C,
                                       float eps, int act_fp32, cudaStream_t st) {
     if (n_rows <= 0 || C <= 0 || !x || !w || !out) return LLARK_EINVAL;
@@ -1104,7 +1316,7 @@ extern "C" int llark_seq_relu2(const void* u, void* y, long long n, int act_fp32
 
 template <typename T, typename TC>
 static void launch_rows(const void* A, long long lda, const void* W, long long ldw, void* C, long long ldc,
-                        const float* bias, int M, int N, int K, int act, cudaStream_t st) {
+                        const float* bias, int M, int N, int K, ActArg act, cudaStream_t st) {
     const int vec = 16 / (int)sizeof(T);
     const int vec_ok = (K % vec == 0) && (lda % vec == 0) && (ldw % vec == 0) &&
                        (((reinterpret_cast<uintptr_t>(A) | reinterpret_cast<uintptr_t>(W)) & 15) == 0);
@@ -1112,7 +1324,7 @@ static void launch_rows(const void* A, long long lda, const void* W, long long l
     // one or two rows: two columns per warp once that still leaves several warps per SM (148 SMs), one for narrow outputs.
     // More rows: blocks of two rows and always two columns (the later row blocks read the weights from L2; a wider row block
     // costs more in registers, and so in warps, than it saves)
-    const bool two = M > 2 || (long long)N >= 2LL * warps * 148 * 2 || act == LLARK_ACT_RELU_GLU;  // (a gate and its up column)
+    const bool two = M > 2 || (long long)N >= 2LL * warps * 148 * 2 || paired(act.kind);  // (a gate and its up column)
     const int nc = two ? 2 : 1;
     const unsigned gx = (unsigned)((N + warps * nc - 1) / (warps * nc));
 #define LLARK_ROWS(MB_, NC_)                                                                                            \
@@ -1124,11 +1336,12 @@ static void launch_rows(const void* A, long long lda, const void* W, long long l
 }
 
 extern "C" int llark_linear_rows(const void* A, long long lda, const void* W, long long ldw, void* C, long long ldc,
-                                 int c_fp32, const float* bias, int M, int N, int K, int in_fp32, int act,
-                                 cudaStream_t st) {
-    if (M <= 0 || N <= 0 || K <= 0 || !A || !W || !C || lda < K || ldw < K || bad_act(act, N) || ldc < out_cols(act, N))
+                                 int c_fp32, const float* bias, int M, int N, int K, int in_fp32, int act_kind,
+                                 float act_limit, float act_slope, cudaStream_t st) {
+    if (M <= 0 || N <= 0 || K <= 0 || !A || !W || !C || lda < K || ldw < K || bad_act(act_kind, N) || ldc < out_cols(act_kind, N))
         return LLARK_EINVAL;
     if (in_fp32 && !c_fp32) return LLARK_EINVAL;
+    const ActArg act{act_kind, act_limit, act_slope};
     if (in_fp32)
         launch_rows<float, float>(A, lda, W, ldw, C, ldc, bias, M, N, K, act, st);
     else if (c_fp32)
@@ -1139,11 +1352,12 @@ extern "C" int llark_linear_rows(const void* A, long long lda, const void* W, lo
 }
 
 extern "C" int llark_linear_simt(const void* A, long long lda, const void* W, long long ldw, void* C, long long ldc,
-                                 int c_fp32, const float* bias, int M, int N, int K, int in_fp32, int act,
-                                 cudaStream_t st) {
-    if (M <= 0 || N <= 0 || K <= 0 || !A || !W || !C || lda < K || ldw < K || bad_act(act, N) || ldc < out_cols(act, N))
+                                 int c_fp32, const float* bias, int M, int N, int K, int in_fp32, int act_kind,
+                                 float act_limit, float act_slope, cudaStream_t st) {
+    if (M <= 0 || N <= 0 || K <= 0 || !A || !W || !C || lda < K || ldw < K || bad_act(act_kind, N) || ldc < out_cols(act_kind, N))
         return LLARK_EINVAL;
     if (in_fp32 && !c_fp32) return LLARK_EINVAL;
+    const ActArg act{act_kind, act_limit, act_slope};
     dim3 grid((N + 63) / 64, (M + 63) / 64);
     if (in_fp32)
         linear_simt_kernel<float, float><<<grid, 256, 0, st>>>((const float*)A, lda, (const float*)W, ldw, (float*)C, ldc,
@@ -1172,10 +1386,10 @@ extern "C" int llark_linear_simt_w32(const void* A, long long lda, const float* 
     dim3 grid((N + 63) / 64, (M + 63) / 64);
     if (in_fp32)
         linear_simt_kernel<float, float, float><<<grid, 256, 0, st>>>((const float*)A, lda, W, ldw, C, ldc, bias, M, N, K,
-                                                                     LLARK_ACT_NONE);
+                                                                     ActArg{LLARK_ACT_NONE, 0.f, 0.f});
     else
         linear_simt_kernel<bf16_t, float, float><<<grid, 256, 0, st>>>((const bf16_t*)A, lda, W, ldw, C, ldc, bias, M, N,
-                                                                      K, LLARK_ACT_NONE);
+                                                                      K, ActArg{LLARK_ACT_NONE, 0.f, 0.f});
     return check_launch();
 }
 

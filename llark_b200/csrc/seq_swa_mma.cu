@@ -47,7 +47,7 @@ swa_mma_kernel(const bf16_t* __restrict__ qn, const bf16_t* __restrict__ kn, con
                long long gate_ld, const float* __restrict__ scale_h, bf16_t* __restrict__ out,
                const int* __restrict__ cu, const int* __restrict__ pos0, const int* __restrict__ slot, int H, int G,
                int D, int window, int cap, const float* __restrict__ sink, int gate_per_head, int chunk, float softcap,
-               const float* __restrict__ vfreq, int v_interleaved) {
+               const float* __restrict__ vfreq, int v_interleaved, long long out_ld, float out_scale) {
     const int b = blockIdx.z, h = blockIdx.y;
     const int g = h / (H / G);
     const int row0 = cu[b], n = cu[b + 1] - row0;
@@ -263,7 +263,7 @@ swa_mma_kernel(const bf16_t* __restrict__ qn, const bf16_t* __restrict__ kn, con
         if (qt0 + r >= n) continue;
         const long long trow = row0 + qt0 + r;
         // a sink adds exp(sink_h) to the denominator (m is in units of log2; every row has seen its own key, so m is finite)
-        const float inv = 1.0f / (sink ? l[x] + exp2f(sink[h] * kLog2e - m[x]) : l[x]);
+        const float inv = out_scale / (sink ? l[x] + exp2f(sink[h] * kLog2e - m[x]) : l[x]);
         const float gh = (gate && gate_per_head) ? 1.0f / (1.0f + expf(-gate[trow * gate_ld + h])) : 1.0f;
         if (vfreq) {
             // Values were stored rotated by their own position: the row's weighted sum is turned back by the query's
@@ -306,7 +306,7 @@ swa_mma_kernel(const bf16_t* __restrict__ qn, const bf16_t* __restrict__ kn, con
                     v0 *= 1.0f / (1.0f + expf(-gp[0]));
                     v1 *= 1.0f / (1.0f + expf(-gp[1]));
                 }
-                *reinterpret_cast<uint32_t*>(out + (trow * H + h) * D + c) = pack_bf16x2(v0, v1);
+                *reinterpret_cast<uint32_t*>(out + trow * out_ld + h * D + c) = pack_bf16x2(v0, v1);
             }
         }
     }
@@ -316,7 +316,8 @@ template <int DMAX>
 static int launch(const void* qn, const void* kn, const void* vv, const void* kring, const void* vring,
                   const float* gate, long long gate_ld, const float* scale_h, void* out, const int* cu, const int* pos0,
                   const int* slot, int n_seq, int max_len, int H, int G, int D, int window, int cap, const float* sink,
-                  int gate_per_head, int chunk, float softcap, const float* vfreq, int v_interleaved, cudaStream_t st) {
+                  int gate_per_head, int chunk, float softcap, const float* vfreq, int v_interleaved, long long out_ld,
+                  float out_scale, cudaStream_t st) {
     const size_t smem = sizeof(bf16_t) * (size_t)(BQ + 4 * BK) * (D + 8);
     if (smem > 48 * 1024) {
         cudaError_t e = cudaFuncSetAttribute(swa_mma_kernel<DMAX>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -329,7 +330,7 @@ static int launch(const void* qn, const void* kn, const void* vv, const void* kr
     swa_mma_kernel<DMAX><<<grid, 128, smem, st>>>((const bf16_t*)qn, (const bf16_t*)kn, (const bf16_t*)vv,
                                                   (const bf16_t*)kring, (const bf16_t*)vring, gate, gate_ld, scale_h,
                                                   (bf16_t*)out, cu, pos0, slot, H, G, D, window, cap, sink, gate_per_head,
-                                                  chunk, softcap, vfreq, v_interleaved);
+                                                  chunk, softcap, vfreq, v_interleaved, out_ld, out_scale);
     cudaError_t e = cudaGetLastError();
     if (e != cudaSuccess) {
         g_last_cuda_error = (int)e;
@@ -347,19 +348,20 @@ extern "C" int llark_seq_swa_attn_mma(const void* qn, const void* kn, const void
                                       const float* gate, long long gate_ld, const float* scale_h, void* out,
                                       const int* cu, const int* pos0, const int* slot, int n_seq, int max_len, int H,
                                       int G, int D, int window, int cap, const float* sink, int gate_per_head,
-                                      int chunk, float softcap, const float* vfreq, int v_interleaved, cudaStream_t st) {
+                                      int chunk, float softcap, const float* vfreq, int v_interleaved, long long out_ld,
+                                      float out_scale, cudaStream_t st) {
     if (n_seq <= 0 || max_len <= 0 || H <= 0 || G <= 0 || (H % G) || D <= 0 || (D % 16) || D > 256 || window <= 0 ||
         cap <= 0 || !qn || !kn || !vv || !kring || !vring || !scale_h || !out || !cu || !pos0 || !slot || chunk < 0 ||
-        softcap < 0.f)
+        softcap < 0.f || out_ld < (long long)H * D || (out_ld % 2))
         return LLARK_EINVAL;
     if (gate && !gate_per_head && (gate_ld % 2)) return LLARK_EINVAL;
     if (vfreq && !v_interleaved && D != 64 && D != 128 && D != 256) return LLARK_EINVAL;
     if (D <= 64)
         return swamma::launch<64>(qn, kn, vv, kring, vring, gate, gate_ld, scale_h, out, cu, pos0, slot, n_seq, max_len, H,
-                                  G, D, window, cap, sink, gate_per_head, chunk, softcap, vfreq, v_interleaved, st);
+                                  G, D, window, cap, sink, gate_per_head, chunk, softcap, vfreq, v_interleaved, out_ld, out_scale, st);
     if (D <= 128)
         return swamma::launch<128>(qn, kn, vv, kring, vring, gate, gate_ld, scale_h, out, cu, pos0, slot, n_seq, max_len,
-                                   H, G, D, window, cap, sink, gate_per_head, chunk, softcap, vfreq, v_interleaved, st);
+                                   H, G, D, window, cap, sink, gate_per_head, chunk, softcap, vfreq, v_interleaved, out_ld, out_scale, st);
     return swamma::launch<256>(qn, kn, vv, kring, vring, gate, gate_ld, scale_h, out, cu, pos0, slot, n_seq, max_len, H, G,
-                               D, window, cap, sink, gate_per_head, chunk, softcap, vfreq, v_interleaved, st);
+                               D, window, cap, sink, gate_per_head, chunk, softcap, vfreq, v_interleaved, out_ld, out_scale, st);
 }

@@ -33,6 +33,9 @@ the same packed weights and stores of its own.
     "relu_glu"   ReluGluFF              down(relu(gate x) * (up x)), one GEMM with the product in its epilogue
     "moe_top_softmax"  TopSoftmaxExperts  biased router, the largest logits are chosen, weights = softmax over those logits;
                                         experts (and an optional shared expert that every token uses) are relu(up x)^2 units
+    "moe_sigmoid_input"  SigmoidInputExperts  the largest logits are chosen, weights = their sigmoids, not renormalised; a weight
+                                        multiplies its expert's INPUT and the outputs are added as they are; experts (and an
+                                        optional shared one with sizes and limit of its own) are clamped gated units
 
     "rotary_attention"  RotaryAttention   grouped-query softmax attention with rotary positions on q and k (halves or
                                         interleaved pairs, part of the head, optionally rescaled frequencies), optional
@@ -45,6 +48,12 @@ the same packed weights and stores of its own.
                                         its own root mean square, no gate; `kv_from` in its configuration: the layer has no
                                         keys and values of its own and reads those of an earlier layer (its stores, and what
                                         the current step brought)
+    "rotary_attention_window"  WindowRotaryAttention   rotary_attention with interleaved pairs, a sliding window, no biases, no gate
+    "retention"  Retention              linear attention with a fixed decay per head, S <- decay S + k v^T, o = S^T q: rotary
+                                        halves on q and k, k / sqrt(dim), every head of o divided by its root mean square, SiLU gate
+    "lightning"  LightningAttention     the same recurrence on SiLU'd q, k and v; o RMS-normed over all heads together, sigmoid gate
+    "parallel_weighted"  WeightedParallelMixers   a rotary_attention_window ("left") and a lightning ("right") side by side on the
+                                        same input, a number weighing each; one input and one output projection for both
     "latent_attention_causal"  LatentCausalAttention   latent attention over everything before (per-position store), rotary
                                         halves, one gate per head
 
@@ -192,12 +201,17 @@ class ReluSquaredFF:
         return {"y": self.forward(x_act)}
 
 
+def _paired_rows(gate, up):
+    """Gate and up rows alternating: what the activations over pairs of columns take."""
+    return torch.stack([gate, up], dim=1).reshape(2 * gate.shape[0], gate.shape[1]).contiguous()
+
+
 class ReluGluFFWeights:
     def __init__(self, w, pfx, spec, width, dev, act):
         F = int(spec["ff"])
         gate, up, self.w_down = (_mat(w, pfx + n, dev, act) for n in ("gate", "up", "down"))
         _expect(pfx, ((gate, (F, width)), (up, (F, width)), (self.w_down, (width, F))))
-        self.w_gu = torch.stack([gate, up], dim=1).reshape(2 * F, width).contiguous()  # rows alternate gate, up
+        self.w_gu = _paired_rows(gate, up)
 
 
 class ReluGluFF:
@@ -641,6 +655,11 @@ class RotaryAttention(_OneBranch):
         w = self.w
         pin = ops.linear(hc, w.w_in, bias=w.b_in, out_dtype=F32)
         self.side = pin[:, :w.side_n] if w.side_n else None
+        return ops.linear(self.attend(pin, st, cache), w.w_o, out_dtype=F32)
+
+    def attend(self, pin, st, cache, out=None, out_scale=1.0):
+        """The heads' outputs (times out_scale) from the fused projection pin; into `out` when given."""
+        w = self.w
         kring, vring = cache.view(self.h_k), cache.view(self.h_v)
         cap = self.ring if self.ring is not None else cache.positions
         single = st.max_len == 1
@@ -658,11 +677,11 @@ class RotaryAttention(_OneBranch):
         o = ops.seq_swa_attn(q, k, v, kring, vring, pin[:, w.g_off:w.n_in] if w.gated else None,
                              pin.stride(0) if w.gated else 0, w.scale_h, st, w.H, w.G, w.D, w.E, window, cap,
                              from_ring_only=single, sink=w.sink, chunk=chunk, softcap=w.softcap, vfreq=w.v_freq,
-                             v_interleaved=w.interleaved)
+                             v_interleaved=w.interleaved, out=out, out_scale=out_scale)
         if own and not single:
             ops.seq_kv_ring_write(k, v, kring, vring, st, cap)
             self.step_kv = (k, v) if self.lends else None
-        return ops.linear(o, w.w_o, out_dtype=F32)
+        return o
 
     def end_step(self):
         """Drops the step's keys and values that other layers may have read."""
@@ -689,6 +708,126 @@ class UnitRotaryAttentionWeights(RotaryAttentionWeights):
 
 class UnitRotaryAttention(RotaryAttention):
     Weights = UnitRotaryAttentionWeights
+
+
+class WindowRotaryAttentionWeights(RotaryAttentionWeights):
+    interleaved = True
+    mask_kind = "window"
+    gated = False
+
+
+class WindowRotaryAttention(RotaryAttention):
+    Weights = WindowRotaryAttentionWeights
+
+
+_FREQUENCIES = {}  # (dims, base, device) -> fp32 tensor: layers with equal rotation share one tensor, and so one table per step
+
+
+def _shared_frequencies(rot, dim, dev, pfx):
+    n = int(rot.get("dims", dim)) if rot else 0
+    if not n:
+        return None
+    if n % 2 or n > dim:
+        raise ValueError(f"{pfx}: rot.dims must be even and at most dim")
+    key = (n, float(rot["base"]), str(dev))
+    if key not in _FREQUENCIES:
+        _FREQUENCIES[key] = rotary_frequencies(n, rot["base"])[0].to(device=dev, dtype=F32).contiguous()
+    return _FREQUENCIES[key]
+
+
+class RetentionWeights:
+    rotates = True      # rotary halves on q and k, k times dim^(-1/2); False: SiLU on q, k and v
+    head_norm = True    # each head of o by its own root mean square, no weight; False: all heads together, weight `norm`
+    gate_silu = True    # SiLU output gate; False: sigmoid
+
+    def __init__(self, w, pfx, spec, width, dev, act):
+        H, D = int(spec["heads"]), int(spec["dim"])
+        E = int(spec.get("vdim", D))
+        self.H, self.D, self.E = H, D, E
+        if len(spec["decay"]) != H:
+            raise ValueError(f"{pfx}: one decay per head")
+        self.powers = ops.decay_powers(spec["decay"], dev)
+        self.freq = _shared_frequencies(spec.get("rot"), D, dev, pfx) if self.rotates else None
+        self.k_scale = D ** -0.5 if self.rotates else 1.0
+        # one projection for q | k | v | gate
+        parts = [_mat(w, pfx + n, dev, act) for n in ("q", "k", "v", "g")]
+        _expect(pfx, [(p, (n, width)) for p, n in zip(parts, (H * D, H * D, H * E, H * E))])
+        self.k_off, self.v_off, self.g_off, self.n_in = H * D, 2 * H * D, 2 * H * D + H * E, 2 * H * D + 2 * H * E
+        self.w_in = _pad_rows(torch.cat(parts))
+        self.norm = None if self.head_norm else _vec(w, pfx + "norm", dev)
+        self.w_o = _mat(w, pfx + "o", dev, act)
+        _expect(pfx, ((self.w_o, (width, H * E)),))
+        if self.norm is not None:
+            _expect(pfx, ((self.norm, (H * E,)),))
+
+
+class Retention(_OneBranch):
+    Weights = RetentionWeights
+
+    def __init__(self, weights, cache, eps, act, max_positions=None):
+        self.w, self.eps, self.act = weights, float(eps), act
+        self.h_state = cache.add_store((weights.H, weights.D, weights.E), F32, zero_on_alloc=True)
+
+    def forward(self, hc, st, cache):
+        w = self.w
+        return ops.linear(self.read_out(ops.linear(hc, w.w_in, out_dtype=F32), st, cache), w.w_o, out_dtype=F32)
+
+    def read_out(self, pin, st, cache, out=None, norm=None):
+        """The gated, normed read-outs from the fused projection pin; into `out` when given. norm: in place of the weight."""
+        w = self.w
+        o = ops.seq_decay_scan(pin, 0, w.k_off, w.v_off, w.powers, cache.view(self.h_state), st, w.H, w.D, w.E, freq=w.freq,
+                               k_scale=w.k_scale, silu=not w.rotates, full_fp32=self.act == F32)
+        H, E = (w.H, w.E) if w.head_norm else (1, w.H * w.E)
+        return ops.seq_head_norm_gate(o, norm if norm is not None else w.norm, H, E, self.eps, self.act,
+                                      gate=pin[:, w.g_off:w.n_in], gate_silu=w.gate_silu, out=out)
+
+
+class LightningAttentionWeights(RetentionWeights):
+    rotates = False
+    head_norm = False
+    gate_silu = False
+
+
+class LightningAttention(Retention):
+    Weights = LightningAttentionWeights
+
+
+class WeightedParallelMixersWeights:
+    def __init__(self, w, pfx, spec, width, dev, act):
+        self.left = WindowRotaryAttentionWeights(w, pfx + "left.", spec["left"], width, dev, act)
+        self.right = LightningAttentionWeights(w, pfx + "right.", spec["right"], width, dev, act)
+        self.left_scale = float(spec["left_scale"])
+        self.right_norm = (self.right.norm * float(spec["right_scale"])).contiguous()  # the right side's number in its norm
+        # both read the same input and their results are added: one projection in (each side's rows are padded to 16-byte
+        # multiples), one out over the two sides' heads side by side
+        self.n_left = self.left.w_in.shape[0]
+        self.w_in = torch.cat([self.left.w_in, self.right.w_in]).contiguous()
+        self.o_left, n_right = self.left.H * self.left.E, self.right.H * self.right.E
+        self.o_right = self.o_left + (-self.o_left) % 8  # the right side starts on a 16-byte boundary
+        self.n_out = self.o_right + n_right
+        self.w_o = torch.zeros((width, self.n_out), device=dev, dtype=act)
+        self.w_o[:, :self.o_left] = self.left.w_o
+        self.w_o[:, self.o_right:] = self.right.w_o
+        self.left.w_in = self.left.w_o = self.right.w_in = self.right.w_o = None  # held once
+
+
+class WeightedParallelMixers(_OneBranch):
+    Weights = WeightedParallelMixersWeights
+
+    def __init__(self, weights, cache, eps, act, max_positions=None):
+        self.w, self.act = weights, act
+        self.left = WindowRotaryAttention(weights.left, cache, eps, act, max_positions)
+        self.right = LightningAttention(weights.right, cache, eps, act, max_positions)
+
+    def forward(self, hc, st, cache):
+        w = self.w
+        pin = ops.linear(hc, w.w_in, out_dtype=F32)
+        heads = torch.empty((st.n_tok, w.n_out), device=hc.device, dtype=self.act)
+        if w.o_right > w.o_left:
+            heads[:, w.o_left:w.o_right].zero_()
+        self.left.attend(pin[:, :w.n_left], st, cache, out=heads[:, :w.o_left], out_scale=w.left_scale)
+        self.right.read_out(pin[:, w.n_left:], st, cache, out=heads[:, w.o_right:], norm=w.right_norm)
+        return ops.linear(heads, w.w_o, out_dtype=F32)
 
 
 class StateSpaceDualityWeights:
@@ -775,7 +914,7 @@ class ClampedGluFFWeights:
         gate, up = _mat(w, pfx + "gate", dev, act), _mat(w, pfx + "up", dev, act)
         self.w_down = _mat(w, pfx + "down", dev, act)
         _expect(pfx, ((gate, (F, width)), (up, (F, width)), (self.w_down, (width, F))))
-        self.w_gu = torch.cat([gate, up]).contiguous()
+        self.w_gu = _paired_rows(gate, up)
 
 
 class ClampedGluFF:
@@ -785,8 +924,11 @@ class ClampedGluFF:
         self.w, self.act = weights, act
 
     def forward(self, x_act):
-        gu = ops.linear(x_act, self.w.w_gu, out_dtype=self.act)
-        return ops.linear(ops.seq_glu_clamped(gu, self.w.limit), self.w.w_down, out_dtype=F32)
+        h = ops.linear(x_act, self.w.w_gu, out_dtype=self.act, act="clamp_glu", act_limit=self.w.limit)
+        return ops.linear(h, self.w.w_down, out_dtype=F32)
+
+    def terms(self, x_act):
+        return {"y": self.forward(x_act)}
 
     def post_norm(self, x, x_act, alpha, w_norm, eps, act):
         """rmsnorm(alpha x + ff(x)) * w_norm -> (fp32, copy in act)."""
@@ -797,6 +939,8 @@ class RoutedExpertsWeights:
     softmax_bias = False  # True: softmax scores, choice on score + `correction`, plain scores as weights
     top_softmax = False   # True: logits with a bias (`router.b`), choice on the logits, softmax over the chosen ones
     gated = True          # experts are down(silu(gate x) * (up x)); False: down(relu(up x)^2)
+    clamped = False       # experts (and the shared one) are clamped gated units with the limits of the configuration
+    sigmoid_input = False  # choice on the logits, weights = their sigmoids as they are, applied to the experts' inputs
 
     def __init__(self, w, pfx, spec, width, dev, act):
         r = spec["router"]
@@ -824,7 +968,9 @@ class RoutedExpertsWeights:
             if self.router_act is not None:
                 self.router_bias = torch.cat([self.router_bias, torch.zeros(pad, device=dev, dtype=F32)]).contiguous()
         names = ("gate", "up") if self.gated else ("up",)
-        self.w_up = torch.stack([torch.cat([_mat(w, f"{pfx}e{e}.{n}", dev, act) for n in names])
+        self.limit = float(spec["expert"]["limit"]) if self.clamped else None
+        pack = (lambda p: _paired_rows(*p)) if self.clamped else torch.cat
+        self.w_up = torch.stack([pack([_mat(w, f"{pfx}e{e}.{n}", dev, act) for n in names])
                                  for e in range(self.n)]).contiguous()
         self.w_down = torch.stack([_mat(w, f"{pfx}e{e}.down", dev, act) for e in range(self.n)]).contiguous()
         self.correction = _vec(w, pfx + "correction", dev) if self.softmax_bias else None
@@ -832,9 +978,10 @@ class RoutedExpertsWeights:
                       (self.w_down, (self.n, width, ff))))
         self.shared = None
         if spec.get("shared"):  # one more expert that every token uses, of a size of its own
-            if self.gated:
-                raise ValueError(f"{pfx}: a shared expert is a squared-ReLU unit")
-            self.shared = ReluSquaredFFWeights(w, pfx + "shared.", spec["shared"], width, dev, act)
+            if self.gated and not self.clamped:
+                raise ValueError(f"{pfx}: a shared expert is a squared-ReLU or a clamped gated unit")
+            unit = ClampedGluFFWeights if self.clamped else ReluSquaredFFWeights
+            self.shared = unit(w, pfx + "shared.", spec["shared"], width, dev, act)
         if self.correction is not None:
             _expect(pfx, ((self.correction, (n_all,)),))
 
@@ -845,7 +992,8 @@ class RoutedExperts:
 
     def __init__(self, weights, act):
         self.w, self.act = weights, act
-        self.shared = ReluSquaredFF(weights.shared, act) if weights.shared is not None else None
+        unit = ClampedGluFF if weights.clamped else ReluSquaredFF
+        self.shared = unit(weights.shared, act) if weights.shared is not None else None
 
     def route(self, x_act):
         w = self.w
@@ -853,27 +1001,31 @@ class RoutedExperts:
             logits = ops.linear(x_act, w.router_act, bias=w.router_bias, out_dtype=F32)[:, :w.n_all]
         else:
             logits = ops.linear_w32(x_act, w.router, bias=w.router_bias)
-        if w.top_softmax:
-            return ops.seq_moe_route_top(logits, w.top)
+        if w.top_softmax or w.sigmoid_input:
+            return ops.seq_moe_route_top(logits, w.top, sigmoid=w.sigmoid_input)
         return ops.seq_moe_route(logits, w.n_groups, w.keep, w.top, w.scale, softmax_bias=w.softmax_bias,
                                  correction=w.correction)
 
-    def experts(self, x_act, ids):
+    def experts(self, x_act, ids, in_wts=None):
         w = self.w
-        return ops.seq_moe_experts(x_act, ids, w.w_up, w.w_down, n_through=w.n_id, gated=w.gated)
+        return ops.seq_moe_experts(x_act, ids, w.w_up, w.w_down, n_through=w.n_id, gated=w.gated, in_wts=in_wts, limit=w.limit)
 
     def terms(self, x_act):
         w = self.w
         if w.n_id:
             raise ValueError("experts that hand their input through need the norm-after-sum residual (post_norm)")
         ids, wts = self.route(x_act)
+        y = self.shared.forward(x_act) if self.shared is not None else None
+        if w.sigmoid_input:
+            z, pos_of = self.experts(x_act, ids, in_wts=wts)
+            return {"y": y, "z": z, "pos_of": pos_of, "top": w.top}
         z, pos_of = self.experts(x_act, ids)
-        return {"y": self.shared.forward(x_act) if self.shared is not None else None, "z": z, "pos_of": pos_of, "wts": wts}
+        return {"y": y, "z": z, "pos_of": pos_of, "wts": wts}
 
     def residual(self, x, y, x_act):
         """x + (y + experts(x_act)): fp32 residual sum with the mixer's output y."""
         w = self.w
-        if w.n_id or self.shared is not None:
+        if w.n_id or self.shared is not None or w.sigmoid_input:
             raise ValueError("experts that hand their input through, and shared ones, need another residual")
         ids, wts = self.route(x_act)
         z, pos_of = self.experts(x_act, ids)
@@ -883,6 +1035,8 @@ class RoutedExperts:
         """rmsnorm(alpha x + experts(x)) * w_norm -> (fp32, copy in act); the weighted sum over a token's choices is taken
         inside the norm kernel, in the order of the choices."""
         w = self.w
+        if w.sigmoid_input:
+            raise ValueError("weights on the experts' inputs need another residual (terms)")
         ids, wts = self.route(x_act)
         z, pos_of = self.experts(x_act, ids)
         y1 = self.shared.forward(x_act) if self.shared is not None else None
@@ -906,11 +1060,22 @@ class TopSoftmaxExperts(RoutedExperts):
     Weights = TopSoftmaxExpertsWeights
 
 
+class SigmoidInputExpertsWeights(RoutedExpertsWeights):
+    clamped = True
+    sigmoid_input = True
+
+
+class SigmoidInputExperts(RoutedExperts):
+    Weights = SigmoidInputExpertsWeights
+
+
 MIXERS = {"attention": GatedWindowAttention, "hgrn2": GatedLinearRecurrence, "latent_attention": LatentWindowAttention,
           "channel_delta": GatedDeltaRule, "general_delta": GeneralizedDeltaRule, "delta": ScalarGatedDeltaRule,
           "sink_attention": SinkAttention, "ssd": StateSpaceDuality, "parallel": ParallelMixers,
           "rotary_attention": RotaryAttention, "rotary_attention_vrot": ValueRotaryAttention,
-          "rotary_attention_unit": UnitRotaryAttention,
+          "rotary_attention_unit": UnitRotaryAttention, "rotary_attention_window": WindowRotaryAttention,
+          "retention": Retention, "lightning": LightningAttention, "parallel_weighted": WeightedParallelMixers,
           "latent_attention_causal": LatentCausalAttention}
 FEED_FORWARDS = {"dense": ReluSquaredFF, "moe": RoutedExperts, "clamped_glu": ClampedGluFF,
-                 "moe_softmax_bias": BiasedSoftmaxExperts, "relu_glu": ReluGluFF, "moe_top_softmax": TopSoftmaxExperts}
+                 "moe_softmax_bias": BiasedSoftmaxExperts, "relu_glu": ReluGluFF, "moe_top_softmax": TopSoftmaxExperts,
+                 "moe_sigmoid_input": SigmoidInputExperts}

@@ -23,6 +23,7 @@ register_native("Golavik", "llark_b200.models.golavik", "GolavikForCausalLM")
 register_native("Gubulorn", "llark_b200.models.gubulorn", "GubulornForCausalLM")
 register_native("Tokatar", "llark_b200.models.tokatar", "TokatarForCausalLM")
 register_native("Manapel", "llark_b200.models.manapel", "ManapelForCausalLM")
+register_native("Buvesun", "llark_b200.models.buvesun", "BuvesunForCausalLM")
 
 
 def read_config(folder):

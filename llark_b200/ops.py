@@ -9,7 +9,7 @@ import math
 
 import torch
 
-from ._lib import (EPI_NONE, EPI_QUICK_GELU, EPI_RELU2, EPI_RELU_GLU, EPI_ROPE, EPI_SWIGLU_BWD, GemmEpilogue, check,
+from ._lib import (EPI_CLAMP_GLU, EPI_NONE, EPI_QUICK_GELU, EPI_RELU2, EPI_RELU_GLU, EPI_ROPE, EPI_SWIGLU_BWD, GemmEpilogue, check,
                    lib)
 
 BF16 = torch.bfloat16
@@ -49,13 +49,13 @@ def _req(t, dtype=None):
 
 def gemm(a, b, *, a_mn=False, b_mn=False, M=None, N=None, K=None, out=None, out_dtype=None, bias=None,
          residual=None, lda=None, ldb=None, ldc=None, ldr=None, max_ctas=0, quick_gelu=False, rope=None,
-         swiglu_bwd=None, act=None):
+         swiglu_bwd=None, act=None, act_limit=0.0, act_slope=0.0):
     """C[M,N] = A[M,K] @ B[N,K]^T (+bias) (+residual), optionally with one fused epilogue (llark_gemm_ex):
 
     quick_gelu=True            C = quick_gelu(acc + bias)
     rope=(cos, sin, S, cols)   columns [0, cols) rotated per 128-wide head, position = row % S (fused-QKV projection)
     swiglu_bwd=gu              acc is d(act) [M, I]; `out` must be the dgu buffer [M, 2I]: out = (dgate | dup)
-    act="relu2" | "relu_glu"   see linear()
+    act="relu2" | "relu_glu" | "clamp_glu"   see linear()
 
     a: [M,K] (a_mn=False) or [K,M] (a_mn=True); b: [N,K] (b_mn=False) or [K,N] (b_mn=True); row-major with
     leading dimension = last-dim stride unless lda/ldb given. bf16 inputs use kind::f16, fp32 inputs kind::tf32.
@@ -92,14 +92,15 @@ def gemm(a, b, *, a_mn=False, b_mn=False, M=None, N=None, K=None, out=None, out_
         e0.record()
     ep = None
     if quick_gelu:
-        ep = GemmEpilogue(EPI_QUICK_GELU, None, None, 0, 0, 0)
+        ep = GemmEpilogue(EPI_QUICK_GELU, None, None, 0, 0, 0, 0.0, 0.0)
     elif rope is not None:
         cos_t, sin_t, S_rope, cols = rope
-        ep = GemmEpilogue(EPI_ROPE, cos_t.data_ptr(), sin_t.data_ptr(), 0, int(S_rope), int(cols))
+        ep = GemmEpilogue(EPI_ROPE, cos_t.data_ptr(), sin_t.data_ptr(), 0, int(S_rope), int(cols), 0.0, 0.0)
     elif swiglu_bwd is not None:
-        ep = GemmEpilogue(EPI_SWIGLU_BWD, swiglu_bwd.data_ptr(), None, swiglu_bwd.stride(0), 0, 0)
+        ep = GemmEpilogue(EPI_SWIGLU_BWD, swiglu_bwd.data_ptr(), None, swiglu_bwd.stride(0), 0, 0, 0.0, 0.0)
     elif act is not None:
-        ep = GemmEpilogue({"relu2": EPI_RELU2, "relu_glu": EPI_RELU_GLU}[act], None, None, 0, 0, 0)
+        ep = GemmEpilogue({"relu2": EPI_RELU2, "relu_glu": EPI_RELU_GLU, "clamp_glu": EPI_CLAMP_GLU}[act], None, None, 0, 0, 0,
+                          float(act_limit), float(act_slope))
     if ep is None:
         rc = lib().llark_gemm(_p(a), int(a_mn), lda, _p(b), int(b_mn), ldb, _p(out), ldc, int(c_fp32), _p(bias),
                               int(bias_fp32), _p(residual), ldr, M, N, K, int(in_fp32), max_ctas, _stream())
@@ -494,13 +495,16 @@ def linear_rows_pays(M, N, K):
 
 
 LINEAR_STATS = {"rows": 0, "tcgen05": 0, "simt": 0}
-LINEAR_ACTS = {None: 0, "relu2": 1, "relu_glu": 2}
+LINEAR_ACTS = {None: 0, "relu2": 1, "relu_glu": 2, "clamp_glu": 3}
+PAIRED_ACTS = ("relu_glu", "clamp_glu")  # two columns of the product, a gate and its up column, make one of the result
+GLU_SLOPE = 1.702
 
 
-def linear(a, w, bias=None, out_dtype=None, out=None, act=None):
+def linear(a, w, bias=None, out_dtype=None, out=None, act=None, act_limit=0.0, act_slope=GLU_SLOPE):
     """y[M, N] = act(a[M, K] @ w[N, K]^T (+ bias fp32 [N])); a and w both bf16 or both fp32 (true fp32 arithmetic, no TF32);
     output bf16 or fp32. act, applied to the fp32 sums before the one rounding: "relu2" = relu(z)^2; "relu_glu": the rows of
-    w alternate gate, up and y [M, N / 2] = relu(z[:, 2c]) * z[:, 2c + 1]."""
+    w alternate gate, up and y [M, N / 2] = relu(z[:, 2c]) * z[:, 2c + 1]; "clamp_glu": the same with g * sigmoid(act_slope * g)
+    * (u + 1), g = min(z[:, 2c], act_limit), u = z[:, 2c + 1] clamped to -act_limit .. act_limit."""
     _req(a), _req(w)
     if a.dtype != w.dtype:
         raise TypeError("linear: activation and weight dtypes differ")
@@ -510,39 +514,43 @@ def linear(a, w, bias=None, out_dtype=None, out=None, act=None):
     if w.shape[1] != K:
         raise ValueError("linear: inner sizes differ")
     code = LINEAR_ACTS[act]
-    if act == "relu_glu" and N % 2:
+    paired = act in PAIRED_ACTS
+    if paired and N % 2:
         raise ValueError("linear: gate and up rows must come in pairs")
     if out is None:
-        out = torch.empty((M, N // 2 if act == "relu_glu" else N), device=a.device, dtype=out_dtype or a.dtype)
+        out = torch.empty((M, N // 2 if paired else N), device=a.device, dtype=out_dtype or a.dtype)
     c_fp32 = _actf(out.dtype)
     if bias is not None:
         _req(bias, torch.float32)
     vec = 4 if c_fp32 else 8
     rows = M <= LINEAR_ROWS_MAX and (in_fp32 or linear_rows_pays(M, N, K))
-    tc = (not rows and not in_fp32 and not (c_fp32 and act == "relu_glu") and K >= 64 and N >= 64 and K % 8 == 0 and a.stride(0) % 8 == 0
+    tc = (not rows and not in_fp32 and not (c_fp32 and paired) and K >= 64 and N >= 64 and K % 8 == 0 and a.stride(0) % 8 == 0
           and w.stride(0) % 8 == 0 and out.stride(0) % vec == 0 and a.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0
           and out.data_ptr() % 16 == 0)
     if rows or (M <= LINEAR_ROWS_MAX and not tc):
         LINEAR_STATS["rows"] += 1
         check(lib().llark_linear_rows(_p(a), a.stride(0), _p(w), w.stride(0), _p(out), out.stride(0), c_fp32, _p(bias),
-                                      M, N, K, in_fp32, code, _stream()), "linear_rows")
+                                      M, N, K, in_fp32, code, float(act_limit), float(act_slope), _stream()), "linear_rows")
     elif tc:
         LINEAR_STATS["tcgen05"] += 1
-        gemm(a, w, bias=bias, out=out, M=M, N=N, K=K, act=act)
+        gemm(a, w, bias=bias, out=out, M=M, N=N, K=K, act=act, act_limit=act_limit, act_slope=act_slope)
     else:
         LINEAR_STATS["simt"] += 1
         check(lib().llark_linear_simt(_p(a), a.stride(0), _p(w), w.stride(0), _p(out), out.stride(0), c_fp32, _p(bias),
-                                      M, N, K, in_fp32, code, _stream()), "linear_simt")
+                                      M, N, K, in_fp32, code, float(act_limit), float(act_slope), _stream()), "linear_simt")
     return out
 
 
-def seq_embed(ids, st, table, pos_table, scale):
-    """ids int32 [n_tok] -> x fp32 [n_tok, C] = table[id] * scale + pos_table[position]."""
+def seq_embed(ids, st, table, pos_table, scale, copy=False):
+    """ids int32 [n_tok] -> x fp32 [n_tok, C] = table[id] * scale + pos_table[position]; copy: (x, x in the table's dtype)."""
     _req(ids, torch.int32)
     C = table.shape[1]
     x = torch.empty((st.n_tok, C), device=table.device, dtype=torch.float32)
+    xa = torch.empty((st.n_tok, C), device=table.device, dtype=BF16) if copy and table.dtype == BF16 else None
     check(lib().llark_seq_embed(_p(ids), _p(st.tok_seq), _p(st.cu), _p(st.pos0), _p(table), _p(pos_table), float(scale),
-                                _p(x), st.n_tok, C, _actf(table.dtype), _stream()), "seq_embed")
+                                _p(x), _p(xa), st.n_tok, C, _actf(table.dtype), _stream()), "seq_embed")
+    if copy:
+        return x, (xa if xa is not None else x)
     return x
 
 
@@ -588,6 +596,37 @@ def seq_gated_norm_add(x, y, w, eps, gate=None, w_next=None, act=None):
                                          _p(w_next), _p(out), _p(xa), rows, C, float(eps),
                                          _actf(act) if w_next is not None else 0, _stream()), "seq_gated_norm_add")
     return (out, xa) if w_next is not None else out
+
+
+def seq_layer_norm(x, w, eps, act, rows=None):
+    """Layer norm (no offset) of fp32 rows in `act`; rows: int32 row numbers (all when None)."""
+    _req(x, torch.float32), _req(w, torch.float32)
+    n, C = (rows.numel() if rows is not None else x.shape[0]), x.shape[1]
+    out = torch.empty((n, C), device=x.device, dtype=act)
+    check(lib().llark_seq_layer_norm_add(_p(x), _p(rows), None, None, None, None, 0, None, _p(w), None, _p(out), n, C,
+                                         float(eps), _actf(act), _stream()), "seq_layer_norm_add(norm)")
+    return out
+
+
+def seq_layer_norm_add(x, eps, y=None, z=None, pos_of=None, wts=None, top=0, w_post=None, w_next=None, act=None,
+                       keep_sum=True):
+    """o = x + f, or x + layernorm(f) * w_post with w_post, f = y + the chosen experts' rows of z (entries pos_of of a token's
+    `top`; wts [n_tok, top]: weighted; either part may be missing). With `act` also layernorm(o) * w_next in that dtype, or,
+    without w_next, o itself in it. Returns (o, that) -- o is None without keep_sum --, or o alone without `act`."""
+    _req(x, torch.float32)
+    rows, C = x.shape
+    for t in (y, z):
+        if t is not None and (not _req(t, torch.float32).is_contiguous() or t.shape[1] != C):
+            raise ValueError("seq_layer_norm_add: sublayer results must be contiguous and of the stream's width")
+    top = (wts.shape[1] if wts is not None else int(top)) if z is not None else 0
+    out = torch.empty_like(x) if keep_sum or act is None or (w_next is None and act != BF16) else None
+    xa = torch.empty((rows, C), device=x.device, dtype=act) if act is not None and (w_next is not None or act == BF16) else None
+    check(lib().llark_seq_layer_norm_add(_p(x), None, _p(y), _p(z), _p(pos_of), _p(wts), top, _p(w_post), _p(w_next), _p(out),
+                                         _p(xa), rows, C, float(eps), _actf(act) if act is not None else 0, _stream()),
+          "seq_layer_norm_add")
+    if act is None:
+        return out
+    return out, (xa if xa is not None else out)
 
 
 def seq_tanh_norm(x, norm, act, rows=None):
@@ -672,13 +711,17 @@ SWA_MMA_MIN_LEN = 16  # shortest longest-request of a step that goes to the tens
 
 
 def seq_swa_attn(qn, kn, vv, kring, vring, gate, gate_ld, scale_h, st, H, G, D, E, window, cap, from_ring_only, sink=None,
-                 gate_per_head=False, chunk=0, softcap=0.0, vfreq=None, v_interleaved=False):
+                 gate_per_head=False, chunk=0, softcap=0.0, vfreq=None, v_interleaved=False, out=None, out_scale=1.0):
     """Softmax attention of a packed step over the last `window` positions (rings of `cap` entries per slot hold what
     earlier steps brought). sink fp32 [H]: one more term exp(sink_h) of the denominator; gate_per_head: gate [n_tok, H].
     chunk > 0: instead of the window the query sees the earlier positions of its own block of `chunk` positions (blocks
     counted from position 0 of the sequence). softcap > 0: score <- softcap * tanh(score / softcap). vfreq fp32 [E / 2]:
-    the values were stored rotated by their own position; each head's weighted sum is turned back by the query's."""
-    out = torch.empty((st.n_tok, H * E), device=qn.device, dtype=qn.dtype)
+    the values were stored rotated by their own position; each head's weighted sum is turned back by the query's.
+    The result times out_scale goes to `out` [n_tok, H * E] (a column slice is fine) when given."""
+    if out is None:
+        out = torch.empty((st.n_tok, H * E), device=qn.device, dtype=qn.dtype)
+    elif out.shape != (st.n_tok, H * E) or out.stride(1) != 1 or out.dtype != qn.dtype:
+        raise ValueError("seq_swa_attn: out does not fit")
     if sink is not None:
         _req(sink, torch.float32)
     if vfreq is not None:
@@ -686,18 +729,19 @@ def seq_swa_attn(qn, kn, vv, kring, vring, gate, gate_ld, scale_h, st, H, G, D, 
         if vfreq.numel() != E // 2:
             raise ValueError("seq_swa_attn: one frequency per pair of value channels")
     if (qn.dtype == BF16 and not from_ring_only and st.max_len >= SWA_MMA_MIN_LEN and D == E and D % 16 == 0
-            and D <= 256 and (gate is None or gate_per_head or gate_ld % 2 == 0)
+            and D <= 256 and out.stride(0) % 2 == 0 and out.data_ptr() % 4 == 0 and (gate is None or gate_per_head or gate_ld % 2 == 0)
             and (vfreq is None or v_interleaved or D in (64, 128, 256))):
         # prompts and portions: 64-query tiles on the tensor cores; single tokens, fp32 and odd head sizes stay SIMT
         check(lib().llark_seq_swa_attn_mma(_p(qn), _p(kn), _p(vv), _p(kring), _p(vring), _p(gate), gate_ld, _p(scale_h),
                                            _p(out), _p(st.cu), _p(st.pos0), _p(st.slot), st.n_seq, st.max_len, H, G, D,
                                            window, cap, _p(sink), int(gate_per_head), int(chunk), float(softcap or 0.0),
-                                           _p(vfreq), int(v_interleaved), _stream()), "seq_swa_attn_mma")
+                                           _p(vfreq), int(v_interleaved), out.stride(0), float(out_scale), _stream()),
+              "seq_swa_attn_mma")
         return out
     check(lib().llark_seq_swa_attn(_p(qn), _p(kn), _p(vv), _p(kring), _p(vring), _p(gate), gate_ld, _p(scale_h), _p(out),
                                    _p(st.tok_seq), _p(st.cu), _p(st.pos0), _p(st.slot), st.n_tok, H, G, D, E, window, cap,
                                    int(from_ring_only), _p(sink), int(gate_per_head), int(chunk), float(softcap or 0.0),
-                                   _p(vfreq), int(v_interleaved), _actf(qn.dtype), _stream()),
+                                   _p(vfreq), int(v_interleaved), out.stride(0), float(out_scale), _actf(qn.dtype), _stream()),
           "seq_swa_attn")
     return out
 
@@ -760,6 +804,62 @@ def seq_glr_scan(src, q_off, f_off, v_off, lower, state, st, H, D, E):
     check(L.llark_seq_glr_scan(_p(src), src.stride(0), q_off, f_off, v_off, _p(lower), _p(cstate), _p(state), None, _p(o),
                                _p(ch.row0), _p(ch.n), _p(ch.index), _p(ch.last_slot), ch.n_items, H, D, E, _stream()),
           "seq_glr_scan(outputs)")
+    return o
+
+
+# linear attention with a fixed decay per head (csrc/seq_decay.cu)
+DECAY_CHUNK = 256         # rows per work item when a long prompt is scanned in chunks
+DECAY_CHUNK_MIN_LEN = 16  # shortest longest-request of a step that goes to the tensor-core kernel
+
+
+def decay_powers(decay, device):
+    """decay^0 .. decay^DECAY_CHUNK per head, fp32 [H, DECAY_CHUNK + 1] (powers taken in float64)."""
+    d = torch.tensor([float(z) for z in decay], dtype=torch.float64)[:, None]
+    return torch.pow(d, torch.arange(DECAY_CHUNK + 1, dtype=torch.float64)[None, :]).to(device=device, dtype=torch.float32).contiguous()
+
+
+def seq_rotary_table(freq, st):
+    """(cos, sin) of position * frequency for every row of the step, fp32 [n_tok, n_freq, 2]; kept with the step for the other
+    layers (and heads, and passes) that rotate by the same tensor of frequencies."""
+    _req(freq, torch.float32)
+    key = freq.data_ptr()
+    if key not in st.tables:
+        cs = torch.empty((st.n_tok, freq.numel(), 2), device=freq.device, dtype=torch.float32)
+        check(lib().llark_seq_rotary_table(_p(freq), freq.numel(), _p(st.tok_seq), _p(st.cu), _p(st.pos0), _p(cs), st.n_tok,
+                                           _stream()), "seq_rotary_table")
+        st.tables[key] = cs
+    return st.tables[key]
+
+
+def seq_decay_scan(src, q_off, k_off, v_off, powers, state, st, H, D, E, freq=None, interleaved=False, k_scale=1.0, silu=False,
+                   full_fp32=False):
+    """src fp32 [n_tok, ld] (q, k: H*D columns at q_off, k_off; v: H*E at v_off) -> o fp32 [n_tok, H*E] of S <- decay_h S + k v^T,
+    o = S^T q; state fp32 [slots, H, D, E] read and written back; powers: decay_powers(). freq: rotary positions on q and k;
+    k_scale: factor on k; silu: SiLU on q, k and v. Prompts go to the tensor-core kernel (three split TF32 products per
+    product, fp32 accuracy), in three passes over chunks of DECAY_CHUNK rows when there are too few (request, head) pairs to
+    fill the GPU; single tokens, short portions, wide heads and full_fp32 to the token-by-token kernel."""
+    _req(src, torch.float32), _req(state, torch.float32), _req(powers, torch.float32)
+    L = lib()
+    o = torch.empty((st.n_tok, H * E), device=src.device, dtype=torch.float32)
+    n_rot = 2 * freq.numel() if freq is not None else 0
+    head = (_p(src), src.stride(0), q_off, k_off, v_off, _p(seq_rotary_table(freq, st)) if n_rot else None, n_rot,
+            int(interleaved), float(k_scale), int(silu), _p(powers), powers.shape[1])
+    if full_fp32 or st.max_len < DECAY_CHUNK_MIN_LEN or D > 128:
+        check(L.llark_seq_decay_rows(*head, _p(state), _p(state), _p(o), _p(st.cu), _p(st.lens_dev), _p(st.slot), _p(st.slot),
+                                     st.n_seq, st.max_len, H, D, E, _stream()), "seq_decay_rows")
+        return o
+    if st.max_len <= DECAY_CHUNK or st.n_seq * H * ((E + 127) // 128) >= 4 * 148:
+        check(L.llark_seq_decay_chunks(*head, _p(state), _p(state), _p(o), _p(st.cu), _p(st.lens_dev), _p(st.slot), _p(st.slot),
+                                       st.n_seq, H, D, E, _stream()), "seq_decay_chunks")
+        return o
+    ch = st.chunks(DECAY_CHUNK)
+    cstate = torch.empty((ch.n_items, H, D, E), device=src.device, dtype=torch.float32)
+    check(L.llark_seq_decay_chunks(*head, None, _p(cstate), None, _p(ch.row0), _p(ch.n), _p(ch.minus1), _p(ch.inner),
+                                   ch.n_items, H, D, E, _stream()), "seq_decay_chunks(local)")
+    check(L.llark_seq_decay_combine(_p(state), _p(cstate), _p(powers), powers.shape[1], _p(ch.n), _p(ch.seq_item0), _p(st.slot),
+                                    st.n_seq, H, D, E, _stream()), "seq_decay_combine")
+    check(L.llark_seq_decay_chunks(*head, _p(cstate), _p(state), _p(o), _p(ch.row0), _p(ch.n), _p(ch.index), _p(ch.last_slot),
+                                   ch.n_items, H, D, E, _stream()), "seq_decay_chunks(outputs)")
     return o
 
 
@@ -847,14 +947,21 @@ def seq_delta_scan(vec, v, state, st, H, D, E, correct=True):
     return o
 
 
-def seq_head_norm_gate(x, w, H, E, eps, act, gate=None, w_per_head=False, gate_silu=False):
-    """x fp32 [n_tok, H*E]: per-head RMS norm, times w ([E] or [H*E]), times sigmoid(gate fp32 [n_tok, H*E]) (gate_silu:
-    times silu(gate)) -> act."""
-    _req(x, torch.float32), _req(w, torch.float32)
-    out = torch.empty(x.shape, device=x.device, dtype=act)
+def seq_head_norm_gate(x, w, H, E, eps, act, gate=None, w_per_head=False, gate_silu=False, out=None):
+    """x fp32 [n_tok, H*E]: per-head RMS norm, times w ([E] or [H*E]; None: no weight), times sigmoid(gate fp32 [n_tok, H*E])
+    (gate_silu: times silu(gate)) -> act, into `out` (a column slice is fine) when given."""
+    _req(x, torch.float32)
+    if w is not None:
+        _req(w, torch.float32)
+    if not x.is_contiguous() or x.shape[1] != H * E:
+        raise ValueError("seq_head_norm_gate: x must be contiguous [n_tok, H * E]")
+    if out is None:
+        out = torch.empty(x.shape, device=x.device, dtype=act)
+    elif out.shape != x.shape or out.stride(1) != 1 or out.dtype != act:
+        raise ValueError("seq_head_norm_gate: out does not fit")
     check(lib().llark_seq_head_norm_gate(_p(x), _p(w), int(w_per_head), _p(gate), gate.stride(0) if gate is not None else 0,
-                                         _p(out), x.shape[0], H, E, float(eps), int(gate_silu), _actf(act), _stream()),
-          "seq_head_norm_gate")
+                                         _p(out), out.stride(0), x.shape[0], H, E, float(eps), int(gate_silu), _actf(act),
+                                         _stream()), "seq_head_norm_gate")
     return out
 
 
@@ -951,13 +1058,14 @@ def seq_moe_route(logits, n_groups, keep, top, scale, softmax_bias=False, correc
     return ids, wts
 
 
-def seq_moe_route_top(logits, top):
-    """The `top` largest logits of each row: expert numbers int32 [n, top] and weights fp32 [n, top] = softmax over them."""
+def seq_moe_route_top(logits, top, sigmoid=False):
+    """The `top` largest logits of each row: expert numbers int32 [n, top] and weights fp32 [n, top] = softmax over them
+    (sigmoid: the sigmoid of each)."""
     n, n_exp = logits.shape
     ids = torch.empty((n, top), device=logits.device, dtype=torch.int32)
     wts = torch.empty((n, top), device=logits.device, dtype=torch.float32)
     check(lib().llark_seq_moe_route_top(_p(_req(logits, torch.float32)), logits.stride(0), _p(ids), _p(wts), n, n_exp,
-                                        int(top), _stream()), "seq_moe_route_top")
+                                        int(top), int(sigmoid), _stream()), "seq_moe_route_top")
     return ids, wts
 
 
@@ -966,15 +1074,21 @@ def seq_moe_route_top(logits, top):
 MOE_DENSE_MIN_ENTRIES = 2048
 
 
-def seq_moe_experts(x, ids, w_up, w_down, n_through=0, gated=True):
-    """x act [n_tok, C]; ids int32 [n_tok, top]; w_up act [n_exp, 2*ff, C] (gate rows, then up rows; silu(gate x) * (up x))
-    or, not gated, [n_exp, ff, C] (relu(up x)^2); w_down act [n_exp, C, ff] -> (z fp32 [n_tok*top, C] expert outputs in sorted order, pos_of int32 [n_tok*top]).
+def seq_moe_experts(x, ids, w_up, w_down, n_through=0, gated=True, in_wts=None, limit=None, slope=GLU_SLOPE):
+    """x act [n_tok, C]; ids int32 [n_tok, top]; w_up act [n_exp, 2*ff, C] (gate rows, then up rows; silu(gate x) * (up x)),
+    with `limit` [n_exp, 2*ff, C] (gate and up rows alternate; the clamped gated unit of linear()'s "clamp_glu"), or, not gated,
+    [n_exp, ff, C] (relu(up x)^2); in_wts fp32 [n_tok, top]: a choice's input is multiplied by its weight; w_down act [n_exp, C, ff] -> (z fp32 [n_tok*top, C] expert outputs in sorted order, pos_of int32 [n_tok*top]).
     n_through: expert numbers n_exp .. n_exp + n_through - 1 have no weights; their rows of z are not written."""
     L = lib()
     n_tok, top = ids.shape
     n_real, n_up, C = w_up.shape
     n_exp = n_real + int(n_through)
+    clamp = limit is not None
+    gated = bool(gated) or clamp
     ff = n_up // 2 if gated else n_up
+    lim, slp = (float(limit), float(slope)) if clamp else (0.0, 0.0)
+    if in_wts is not None and (_req(in_wts, torch.float32).shape != ids.shape or not in_wts.is_contiguous()):
+        raise ValueError("seq_moe_experts: one weight per choice")
     n_ent = n_tok * top
     dense = (x.dtype == BF16 and n_ent >= MOE_DENSE_MIN_ENTRIES and C % 8 == 0 and ff % 8 == 0 and C >= 64 and ff >= 64
              and L.llark_gemm_get_mode() == 1)
@@ -999,17 +1113,21 @@ def seq_moe_experts(x, ids, w_up, w_down, n_through=0, gated=True):
             init()
         count = meta[1:]
         xs = torch.empty((n_ent, C), device=x.device, dtype=x.dtype)
-        check(L.llark_seq_moe_gather(_p(x), x.stride(0), _p(perm), top, _p(xs), n_ent, C, 0, _stream()), "seq_moe_gather")
-        gu = torch.empty((n_ent, n_up), device=x.device, dtype=x.dtype) if gated else act
-        check(L.llark_gemm_segments(_p(xs), C, _p(w_up), _p(gu), n_up, 0, None, n_real, _p(tiles256), max256, _p(count),
-                                    n_ent, n_up, C, EPI_NONE if gated else EPI_RELU2, _stream()), "gemm_segments(up)")
-        if gated:
+        check(L.llark_seq_moe_gather(_p(x), x.stride(0), _p(perm), top, _p(xs), n_ent, C, _p(in_wts), 0, _stream()),
+              "seq_moe_gather")
+        split = gated and not clamp  # gate and up halves apart: their product is a kernel of its own
+        gu = torch.empty((n_ent, n_up), device=x.device, dtype=x.dtype) if split else act
+        epi = EPI_CLAMP_GLU if clamp else (EPI_NONE if gated else EPI_RELU2)
+        check(L.llark_gemm_segments(_p(xs), C, _p(w_up), _p(gu), gu.shape[1], 0, None, n_real, _p(tiles256), max256, _p(count),
+                                    n_ent, n_up, C, epi, lim, slp, _stream()), "gemm_segments(up)")
+        if split:
             check(L.llark_seq_silu_mul(_p(gu), _p(act), n_ent, ff, 0, _stream()), "seq_silu_mul")
         check(L.llark_gemm_segments(_p(act), ff, _p(w_down), _p(z), C, 1, None, n_real, _p(tiles256), max256, _p(count),
-                                    n_ent, C, ff, EPI_NONE, _stream()), "gemm_segments(down)")
+                                    n_ent, C, ff, EPI_NONE, 0.0, 0.0, _stream()), "gemm_segments(down)")
         return z, pos_of
     check(L.llark_seq_moe_up(_p(x), x.stride(0), _p(perm), top, _p(w_up), _p(act), _p(tiles), _p(meta), max_tiles,
-                             n_ent, ff, C, int(gated), _actf(x.dtype), _stream()), "seq_moe_up")
+                             n_ent, ff, C, 2 if clamp else int(gated), _p(in_wts), lim, slp, _actf(x.dtype), _stream()),
+          "seq_moe_up")
     check(L.llark_seq_moe_down(_p(act), _p(w_down), _p(z), _p(tiles), _p(meta), max_tiles, n_ent, C, ff, _actf(x.dtype),
                                _stream()), "seq_moe_down")
     return z, pos_of

@@ -60,7 +60,7 @@ def parse():
     ap.add_argument("--no-torch-baseline", action="store_true",
                     help="skip the stock-PyTorch run of the reference's model class on the same GPU (N=1 only)")
     ap.add_argument("--workload", default="llama", choices=["llama", "e2e", "generation", "generation-golavik", "generation-gubulorn", "generation-tokatar",
-                                                                  "generation-manapel"],
+                                                                  "generation-manapel", "generation-buvesun"],
                     help="llama = BASELINE configs[2] (precomputed Jukebox embeds, the default headline); "
                          "e2e = configs[3]: 25 s waveform -> Jukebox front end -> projector -> Llama step in-process; "
                          "generation = prefill / decode tokens/s of the Kelutar decoder beside the Llama path at equal "
@@ -69,7 +69,8 @@ def parse():
                          "generation-gubulorn = the same for the Gubulorn decoder beside Golavik at equal size; "
                          "generation-tokatar = the same for the Tokatar decoder beside an all-attention Kelutar at equal size; "
                          "generation-manapel = the same for the Manapel decoder beside an all-attention Tokatar and a Golavik "
-                         "with the same experts")
+                         "with the same experts; "
+                         "generation-buvesun = the same for the Buvesun decoder beside Gubulorn and Kelutar at equal size")
     ap.add_argument("--jukebox-precision", default="bf16", choices=["bf16", "tf32"])
     return ap.parse_args()
 
@@ -634,6 +635,13 @@ def main():
         torch.cuda.set_device(int(os.environ.get("LOCAL_RANK", "0")))
         pk, kind = peaks()
         bench_generation.run_manapel(args, pk, kind, emit)
+        return
+    if args.workload == "generation-buvesun":
+        from llark_b200 import bench_generation
+
+        torch.cuda.set_device(int(os.environ.get("LOCAL_RANK", "0")))
+        pk, kind = peaks()
+        bench_generation.run_buvesun(args, pk, kind, emit)
         return
     world = int(os.environ.get("WORLD_SIZE", "1"))
     rank = int(os.environ.get("RANK", "0"))

@@ -1,7 +1,7 @@
 """Generation throughput of the Kelutar path beside the Llama path at equal size (`bench.py --workload generation`), of
 Golavik beside Kelutar (`generation-golavik`), of Gubulorn beside Golavik (`generation-gubulorn`), of Tokatar beside an
-all-attention Kelutar (`generation-tokatar`) and of Manapel beside an all-attention Tokatar and a Golavik with the same
-experts (`generation-manapel`).
+all-attention Kelutar (`generation-tokatar`), of Manapel beside an all-attention Tokatar and a Golavik with the same
+experts (`generation-manapel`) and of Buvesun beside Gubulorn and Kelutar (`generation-buvesun`).
 
 Random weights, synthetic token ids. For each size: prefill tokens/s (a packed batch of whole prompts) and decode tokens/s
 (one token per request and step, after a prompt of `context` tokens) for both decoders, plus a per-op table: every op
@@ -116,11 +116,13 @@ def timed(fn, warmup, iters, flush, setup=None):
 
 
 class OpTimer:
-    """Wraps the named functions of llark_b200.ops with CUDA-event brackets while active."""
+    """Wraps the named functions of llark_b200.ops with CUDA-event brackets while active. Bytes and FLOPs are counted at the
+    call, so that the records keep no tensor alive (a step that outgrows the allocator's pool would be timed with it)."""
 
-    def __init__(self, names):
+    def __init__(self, names, ctx=None):
         from llark_b200 import ops
 
+        self.ctx = ctx or {}
         self.ops, self.names, self.saved, self.records, self.depth = ops, names, {}, [], 0
 
     def __enter__(self):
@@ -139,7 +141,8 @@ class OpTimer:
                 finally:
                     self.depth -= 1
                 e1.record()
-                self.records.append((__n, e0, e1, a, k, out))
+                shape = (a[0].shape[0], a[1].shape[0], a[0].shape[1]) if __n == "linear" else None
+                self.records.append((__n, e0, e1, _op_work(__n, a, k, out, self.ctx), shape))
                 return out
 
             setattr(self.ops, n, wrap)
@@ -170,13 +173,14 @@ def _op_work(name, a, k, out, ctx):
     if name == "seq_swa_attn":
         qn, st, H, G, D, E, window = a[0], a[8], a[9], a[10], a[11], a[12], a[13]
         chunk = k.get("chunk") or 0
+        gate = st.n_tok * (H if k.get("gate_per_head") else H * E) * 4 if a[5] is not None else 0
         if chunk:  # a query sees its own block of positions up to itself; the step reads its blocks' keys once
             keys = sum((p0 + i) % chunk + 1 for p0, n in zip(st.pos0_host, st.lens) for i in range(n))
             kv_once = sum(n + min(p0 % chunk, p0) for p0, n in zip(st.pos0_host, st.lens)) * G * (D + E) * 2
-            return 2 * _nbytes(qn) + kv_once + st.n_tok * H * E * 4, 2.0 * keys * H * (D + E)
+            return 2 * _nbytes(qn) + kv_once + gate, 2.0 * keys * H * (D + E)
         keys = sum(min(window, p0 + i + 1) for p0, n in zip(st.pos0_host, st.lens) for i in range(n))
         kv_once = sum(min(n + min(window, p0), n + window) for p0, n in zip(st.pos0_host, st.lens)) * G * (D + E) * 2
-        return 2 * _nbytes(qn) + kv_once + st.n_tok * H * E * 4, 2.0 * keys * H * (D + E)
+        return 2 * _nbytes(qn) + kv_once + gate, 2.0 * keys * H * (D + E)
     if name == "attn_fwd":
         qkv, B, S, NH, D = a[0], a[2], a[3], a[4], a[5]
         return _nbytes(qkv) + B * S * NH * D * 2, 4.0 * B * NH * D * S * (S + 1) / 2
@@ -187,6 +191,9 @@ def _op_work(name, a, k, out, ctx):
     if name == "seq_glr_scan":
         src, state, st, H, D, E = a[0], a[5], a[6], a[7], a[8], a[9]
         return _nbytes(src) + 2 * st.n_seq * H * D * E * 4 + st.n_tok * H * E * 4, 5.0 * st.n_tok * H * D * E
+    if name == "seq_decay_scan":  # q, k, v columns in, o out, the state once in and out; decay, write and read-out per entry
+        st, H, D, E = a[6], a[7], a[8], a[9]
+        return (st.n_tok * H * (2 * D + 2 * E) * 4 + 2 * st.n_seq * H * D * E * 4), 5.0 * st.n_tok * H * D * E
     if name == "seq_delta_scan":
         vec, v, state, st, H, D, E = a[0], a[1], a[2], a[3], a[4], a[5], a[6]
         per = 9.0 if k.get("correct", True) else 5.0  # without the correction: decay, write and read-out only
@@ -224,14 +231,12 @@ def op_table(records, ctx, peaks):
 
     bw, fl = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
     agg = {}
-    for name, e0, e1, a, k, out in records:
+    for name, e0, e1, (nb, flops), shape in records:
         if name == "gemm" and ctx.get("skip_gemm"):
             continue  # already inside `linear`
         ms = e0.elapsed_time(e1)
-        nb, flops = _op_work(name, a, k, out, ctx)
         if name == "linear":
-            M, K = a[0].shape
-            name = "linear_rows" if M <= 8 and ops.linear_rows_pays(M, a[1].shape[0], K) else "linear_tcgen05"
+            name = "linear_rows" if shape[0] <= 8 and ops.linear_rows_pays(*shape) else "linear_tcgen05"
         if name == "gemm":
             name = "gemm_tcgen05"
         d = agg.setdefault(name, {"calls": 0, "ms": 0.0, "bytes": 0, "flops": 0.0, "roof_ms": 0.0})
@@ -761,6 +766,117 @@ def run_manapel(args, peaks, peaks_kind, emit):
           "sizes": results, "wall_s": round(time.time() - t0, 1)})
 
 
+BUVESUN_OPS = ["linear", "linear_w32", "seq_embed", "seq_layer_norm", "seq_layer_norm_add", "seq_rotary_table", "seq_decay_scan",
+               "seq_head_norm_gate", "seq_qkv_rotary", "seq_swa_attn", "seq_kv_ring_write", "seq_moe_route_top", "seq_moe_experts"]
+
+# (name, width, layer runs, heads, key/value heads, head dim, window, experts, top, expert ff, shared ff, vocab): one retention
+# layer that runs in half of the places (a loop), parallel layers in the others, experts everywhere. Beside it: a Gubulorn
+# model with as many layers of the same width, heads and experts, and a Kelutar model of as many layers (three recurrences to
+# one window attention of the same heads; a feed-forward of top x expert ff rows on the attention layers).
+BUVESUN_SIZES = [
+    ("b2048", 2048, 4, 16, 4, 128, 1024, 32, 4, 1024, 2048, 32000),
+    ("b4096", 4096, 4, 32, 8, 128, 2048, 64, 6, 1024, 2048, 32000),
+]
+
+
+def buvesun_config(width, runs, heads, kv, dim, window, experts, top, ff, shared, vocab):
+    mlp = {"kind": "moe", "expert": {"ff": ff, "limit": 7.0}, "router": {"experts": experts, "top": top},
+           "shared": {"ff": shared, "limit": 7.0}}
+    decay = [1.0 - 2.0 ** (-5 - 7.0 * h / max(heads - 1, 1)) for h in range(heads)]
+    memory = {"heads": heads, "dim": dim, "vdim": dim, "decay": decay}
+    ret = {"type": "retention", "mixer": dict(memory, rot={"base": 10000.0, "dims": dim}), "mlp": mlp}
+    par = {"type": "parallel", "mlp": mlp,
+           "mixer": {"left": {"heads": heads, "kv_heads": kv, "dim": dim, "vdim": dim, "scale": 1.0 / math.sqrt(dim),
+                              "mask": {"size": window}, "rot": {"base": 10000.0, "dims": dim}},
+                     "right": memory, "left_scale": 0.7, "right_scale": 0.6}}
+    return {"architecture": "Buvesun", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+            "residual_mult": 0.5, "loop": {"start": 0, "stop": 1, "times": runs // 2}, "layers": [ret] + [par] * (runs - runs // 2)}
+
+
+def buvesun_random_weights(cfg, device, seed=0):
+    g = torch.Generator(device=device).manual_seed(seed)
+    C = cfg["width"]
+
+    def mat(o, i, s=None):
+        return (torch.randn(o, i, device=device, generator=g) * (s or 1.0 / math.sqrt(i))).to(BF16)
+
+    def vec(n, mean=1.0, s=0.1):
+        return (mean + torch.randn(n, device=device, generator=g) * s).to(BF16)
+
+    W = {"embed": mat(cfg["vocab"], C, 1.0), "head": mat(cfg["vocab"], C), "final.norm": vec(C), "loop.in": mat(C, 2 * C)}
+    for i, layer in enumerate(cfg["layers"]):
+        p, m, mlp = "l%d." % i, layer["mixer"], layer["mlp"]
+        for n in ("norm1", "norm1b", "ls1", "norm2", "norm2b", "ls2"):
+            W[p + n] = vec(C)
+        memories = [("mix.", m)]
+        if layer["type"] == "parallel":
+            a = m["left"]
+            rows = {"q": a["heads"] * a["dim"], "k": a["kv_heads"] * a["dim"], "v": a["kv_heads"] * a["vdim"]}
+            W.update({p + "mix.left." + n: mat(r, C) for n, r in rows.items()})
+            W[p + "mix.left.o"] = mat(C, a["heads"] * a["vdim"])
+            memories = [("mix.right.", m["right"])]
+            W[p + "mix.right.norm"] = vec(m["right"]["heads"] * m["right"]["vdim"])
+        for x, b in memories:
+            hd, he = b["heads"] * b["dim"], b["heads"] * b["vdim"]
+            W.update({p + x + "q": mat(hd, C), p + x + "k": mat(hd, C), p + x + "v": mat(he, C), p + x + "g": mat(he, C),
+                      p + x + "o": mat(C, he)})
+        n = mlp["router"]["experts"]
+        W[p + "mlp.router"] = mat(n, C)
+        units = {"e%d." % e: mlp["expert"]["ff"] for e in range(n)}
+        units["shared."] = mlp["shared"]["ff"]
+        for u, f in units.items():
+            W.update({p + "mlp." + u + "gate": mat(f, C), p + "mlp." + u + "up": mat(f, C), p + "mlp." + u + "down": mat(C, f)})
+    return W
+
+
+def bench_size_buvesun(name, width, runs, heads, kv, dim, window, experts, top, ff, shared, vocab, peaks, steps, warmup,
+                       prefill_batch=4, prompt=2048, decode_batches=(1, 8, 32), context=1024):
+    """Buvesun beside the two existing decoders that share its parts: Gubulorn (attention beside a recurrence, clamped gated
+    units, routed experts) and Kelutar (linear recurrences and window attention)."""
+    from llark_b200.models.buvesun import BuvesunConfig, BuvesunForCausalLM
+    from llark_b200.models.gubulorn import GubulornConfig, GubulornForCausalLM
+    from llark_b200.models.kelutar import KelutarConfig, KelutarForCausalLM
+
+    flush = _Flush()
+    out = {"size": name, "width": width, "layer_runs": runs, "heads": heads, "kv_heads": kv, "head_dim": dim, "window": window,
+           "experts": experts, "top": top, "expert_ff": ff, "shared_ff": shared, "vocab": vocab,
+           "prefill": {"batch": prefill_batch, "prompt": prompt}, "decode": {"context": context}}
+    g = torch.Generator().manual_seed(0)
+    bcfg = buvesun_config(width, runs, heads, kv, dim, window, experts, top, ff, shared, vocab)
+    ucfg = gubulorn_config(width, runs, heads, dim, experts, 8, top, ff, width // 32, 128, vocab)
+    kcfg = kelutar_config(width, runs, heads, dim, window, top * ff, vocab, max(prompt, context) + 64)
+    for tag, cls, conf, cfg, weights, op_names in (
+            ("buvesun", BuvesunForCausalLM, BuvesunConfig, bcfg, buvesun_random_weights, BUVESUN_OPS),
+            ("gubulorn", GubulornForCausalLM, GubulornConfig, ucfg, gubulorn_random_weights, GUBULORN_OPS),
+            ("kelutar", KelutarForCausalLM, KelutarConfig, kcfg, kelutar_random_weights, KELUTAR_OPS)):
+        m = cls(conf.from_dict(cfg), weights(cfg, "cuda"), dtype=BF16)
+        if m.engine.max_positions is None:
+            m.engine.max_positions = max(prompt, context) + 64
+        bench_native(tag, m.engine, op_names, out, vocab, peaks, steps, warmup, flush, g, prefill_batch, prompt,
+                     decode_batches, context)
+        del m
+        torch.cuda.empty_cache()
+    return out
+
+
+def run_buvesun(args, peaks, peaks_kind, emit):
+    from llark_b200 import ops
+
+    ops.init()
+    t0 = time.time()
+    sizes = [s for s in BUVESUN_SIZES if not os.environ.get("LLARK_BENCH_SIZE") or s[0] == os.environ["LLARK_BENCH_SIZE"]]
+    results = [bench_size_buvesun(*s, peaks=peaks, steps=args.steps, warmup=max(args.warmup, 3)) for s in sizes]
+    head = results[0]
+    emit({"metric": "generation tokens/s, Buvesun beside Gubulorn and Kelutar at equal size (prefill of %d x %d tokens)"
+                    % (head["prefill"]["batch"], head["prefill"]["prompt"]),
+          "value": head["prefill"]["buvesun_tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "steps": args.steps,
+          "warmup": max(args.warmup, 3), "ms_per_step": head["prefill"]["buvesun_ms"], "higher_is_better": True,
+          "scaling": "weak", "vs_baseline": None, "dtype": "bf16", "data": "synthetic token ids, random weights",
+          "config": {"model": "Buvesun " + head["size"], "l2": "256 MB fill between timed steps",
+                     "peaks": peaks_kind, "hbm_gbs": peaks["hbm_gbs"], "bf16_tflops": peaks["bf16_tflops"]},
+          "sizes": results, "wall_s": round(time.time() - t0, 1)})
+
+
 def bench_size(name, width, layers, heads, dim, window, ff, vocab, peaks, steps, warmup, prefill_batch=4,
                prompt=2048, decode_batches=(1, 8, 32), context=1024):
     from llark_b200.models.kelutar import KelutarConfig, KelutarForCausalLM
@@ -836,7 +952,7 @@ def bench_size(name, width, layers, heads, dim, window, ff, vocab, peaks, steps,
         out["decode"]["llama_b%d_ms" % B] = round(ms, 3)
         if B == decode_batches[-1] or B == 8:
             for _ in range(2):
-                with OpTimer(LLAMA_OPS) as t:
+                with OpTimer(LLAMA_OPS, {"context": context}) as t:
                     l_step()
             out["decode"]["llama_b%d_ops" % B] = op_table(t.records, {"context": context}, peaks)
     del lm, le, lc

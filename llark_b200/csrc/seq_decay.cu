@@ -218,51 +218,88 @@ __device__ __forceinline__ void mma3(float (&c)[4], const FragA& a, const FragB&
     mma_tf32(c, a.hi, b.hi[0], b.hi[1]);
 }
 
-// One q or k head of kL rows -> dst [kL][DS]; rows >= cnt and columns >= D are zero. vec: 16-byte pieces are possible.
-__device__ __forceinline__ void load_heads(const DecayIn& in, int off, long long row, int cnt, int h, int D, int Dp, int DS,
-                                           float scale, int vec, float* dst) {
-    const int nq = Dp >> 2;
-    const int half = in.n_rot >> 1;
+// Rows of one head (D entries from column off of src) -> dst [kL][pitch], zero behind the step's rows and behind D, as
+// asynchronous copies of 16 bytes (vec) or of single words.
+__device__ __forceinline__ void copy16(float* dst, const float* src, bool live) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(live ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void copy4(float* dst, const float* src, bool live) {
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(live ? 4 : 0) : "memory");
+}
+__device__ __forceinline__ void fetch_head(const float* src, long long ld, int cnt, int D, int Dp, int pitch, int vec, float* dst) {
+    if (vec) {
+        const int nq = Dp >> 2;
+        for (int i = threadIdx.x; i < kL * nq; i += blockDim.x) {
+            const int tk = i / nq, d = (i % nq) * 4;
+            const bool live = tk < cnt && d < D;
+            copy16(dst + tk * pitch + d, live ? src + tk * ld + d : src, live);
+        }
+    } else {
+        for (int i = threadIdx.x; i < kL * Dp; i += blockDim.x) {
+            const int tk = i / Dp, d = i % Dp;
+            const bool live = tk < cnt && d < D;
+            copy4(dst + tk * pitch + d, live ? src + tk * ld + d : src, live);
+        }
+    }
+}
+// SiLU in the accuracy of the fast exponential and division (about 2^-21 relative), in place over kL rows
+__device__ __forceinline__ float silu_fast(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
+__device__ __forceinline__ void silu_rows(float* x, int width, int pitch) {
+    const int nq = width >> 2;
     for (int i = threadIdx.x; i < kL * nq; i += blockDim.x) {
-        const int tk = i / nq, d = (i % nq) * 4;
-        float* out = dst + tk * DS + d;
-        const bool live = tk < cnt;
-        const long long t = row + tk;
-        const float* x = in.src + t * in.ld + off + (long long)h * D;
-        if (!live || d >= D) {
-            if (in.n_rot && !in.interleaved && vec && d >= half && d < in.n_rot) continue;  // its partner writes it
-            *reinterpret_cast<float4*>(out) = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (in.n_rot && !in.interleaved && vec && d < half)
-                *reinterpret_cast<float4*>(out + half) = make_float4(0.f, 0.f, 0.f, 0.f);
-            continue;
-        }
-        if (!vec) {
-#pragma unroll
-            for (int j = 0; j < 4; ++j) out[j] = d + j < D ? qk_entry(in, x, t, d + j) * scale : 0.f;
-            continue;
-        }
-        float4 a = *reinterpret_cast<const float4*>(x + d);
-        if (in.silu) {
-            a.x = siluf_(a.x), a.y = siluf_(a.y), a.z = siluf_(a.z), a.w = siluf_(a.w);
-        } else if (d < in.n_rot) {
-            if (in.interleaved) {  // pairs (x, y) and (z, w)
-                const float4 c = *reinterpret_cast<const float4*>(in.cs + t * half + (d >> 1));
-                a = make_float4(a.x * c.x - a.y * c.y, a.y * c.x + a.x * c.y, a.z * c.z - a.w * c.w, a.w * c.z + a.z * c.w);
-            } else {
-                if (d >= half) continue;  // written together with the first halves
-                const float4 b = *reinterpret_cast<const float4*>(x + d + half);
-                const float4* cp = reinterpret_cast<const float4*>(in.cs + t * half + d);
-                const float4 c0 = cp[0], c1 = cp[1];  // (cos, sin) of pairs d, d + 1 and d + 2, d + 3
-                const float4 u = make_float4(a.x * c0.x - b.x * c0.y, a.y * c0.z - b.y * c0.w, a.z * c1.x - b.z * c1.y,
-                                             a.w * c1.z - b.w * c1.w);
-                const float4 v = make_float4(b.x * c0.x + a.x * c0.y, b.y * c0.z + a.y * c0.w, b.z * c1.x + a.z * c1.y,
-                                             b.w * c1.z + a.w * c1.w);
-                *reinterpret_cast<float4*>(out + half) = make_float4(v.x * scale, v.y * scale, v.z * scale, v.w * scale);
-                a = u;
+        float4* p = reinterpret_cast<float4*>(x + (i / nq) * pitch + (i % nq) * 4);
+        const float4 v = *p;
+        *p = make_float4(silu_fast(v.x), silu_fast(v.y), silu_fast(v.z), silu_fast(v.w));
+    }
+}
+__device__ __forceinline__ void turn4(float4& u, float4& v, float4 c0, float4 c1, float f) {
+    const float4 a = u, b = v;  // c0, c1: (cos, sin) of four neighbouring pairs (u.x, v.x) .. (u.w, v.w)
+    u = make_float4((a.x * c0.x - b.x * c0.y) * f, (a.y * c0.z - b.y * c0.w) * f, (a.z * c1.x - b.z * c1.y) * f,
+                    (a.w * c1.z - b.w * c1.w) * f);
+    v = make_float4((b.x * c0.x + a.x * c0.y) * f, (b.y * c0.z + a.y * c0.w) * f, (b.z * c1.x + a.z * c1.y) * f,
+                    (b.w * c1.z + a.w * c1.w) * f);
+}
+// Rotation of q (when there is one) and k and the factor on k, in place. A pair belongs to one thread.
+__device__ __forceinline__ void turn_rows(const DecayIn& in, long long row, int cnt, int D, int DS, float* sQ, float* sK) {
+    const int half = in.n_rot >> 1;
+    const float f = in.k_scale;
+    if (half && half % 4 == 0 && !in.interleaved) {
+        const int nq = half >> 2;
+        for (int i = threadIdx.x; i < cnt * nq; i += blockDim.x) {
+            const int tk = i / nq, d = (i % nq) * 4;
+            const float4* cp = reinterpret_cast<const float4*>(in.cs + (row + tk) * half + d);
+            const float4 c0 = __ldg(cp), c1 = __ldg(cp + 1);
+            float4* ku = reinterpret_cast<float4*>(sK + tk * DS + d);
+            float4* kv = reinterpret_cast<float4*>(sK + tk * DS + d + half);
+            float4 u = *ku, v = *kv;
+            turn4(u, v, c0, c1, f);
+            *ku = u, *kv = v;
+            if (sQ) {
+                float4* qu = reinterpret_cast<float4*>(sQ + tk * DS + d);
+                float4* qv = reinterpret_cast<float4*>(sQ + tk * DS + d + half);
+                u = *qu, v = *qv;
+                turn4(u, v, c0, c1, 1.0f);
+                *qu = u, *qv = v;
             }
         }
-        *reinterpret_cast<float4*>(out) = make_float4(a.x * scale, a.y * scale, a.z * scale, a.w * scale);
+    } else {
+        for (int i = threadIdx.x; i < cnt * half; i += blockDim.x) {
+            const int tk = i / half, m = i % half;
+            const int a = tk * DS + (in.interleaved ? 2 * m : m), b = tk * DS + (in.interleaved ? 2 * m + 1 : m + half);
+            const float2 c = in.cs[(row + tk) * half + m];
+            float u = sK[a], v = sK[b];
+            sK[a] = (u * c.x - v * c.y) * f;
+            sK[b] = (v * c.x + u * c.y) * f;
+            if (sQ) {
+                u = sQ[a], v = sQ[b];
+                sQ[a] = u * c.x - v * c.y;
+                sQ[b] = v * c.x + u * c.y;
+            }
+        }
     }
+    const int rest = D - in.n_rot;
+    if (f != 1.0f)
+        for (int i = threadIdx.x; i < cnt * rest; i += blockDim.x) sK[(i / rest) * DS + in.n_rot + i % rest] *= f;
 }
 
 // Block = up to 128 columns (16 per warp) of one head of one work item. A warp keeps its 16 columns of S transposed in
@@ -278,10 +315,8 @@ decay_chunk_kernel(DecayIn in, const float* __restrict__ pow_h, int pow_ld, cons
     constexpr int Dp = 8 * NT, DS = Dp + 8;
     extern __shared__ __align__(16) float sm[];
     const int cols = (blockDim.x >> 5) * 16, VS = cols + 8;
-    float* sQ = sm;
-    float* sK = sQ + kL * DS;
-    float* sV = sK + kL * DS;
-    float* sA = sV + kL * VS;
+    const int stage_floats = kL * (2 * DS + VS);  // two stages of Q | K | V: one is computed on while the other arrives
+    float* sA = sm + 2 * stage_floats;
     float* spw = sA + kL * kAS;  // decay^0 .. decay^kL
     const int h = blockIdx.y, b = blockIdx.z;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarp = blockDim.x >> 5;
@@ -302,27 +337,32 @@ decay_chunk_kernel(DecayIn in, const float* __restrict__ pow_h, int pow_ld, cons
             const int d = 8 * nt + 2 * t4 + (c & 1), e = ew + g + (c >> 1) * 8;
             S[nt][c] = (si && d < D && e < E) ? si[(long long)d * E + e] : 0.f;
         }
-    for (int t0 = 0; t0 < n; t0 += kL) {
+    auto fetch = [&](int t0, float* base) {
+        const int cnt = n - t0 < kL ? n - t0 : kL;
+        const float* r = in.src + (row0 + t0) * in.ld;
+        if (o) fetch_head(r + in.q_off + (long long)h * D, in.ld, cnt, D, Dp, DS, vec, base);
+        fetch_head(r + in.k_off + (long long)h * D, in.ld, cnt, D, Dp, DS, vec, base + kL * DS);
+        fetch_head(r + in.v_off + (long long)h * E + e0, in.ld, cnt, E - e0 < cols ? E - e0 : cols, cols, VS, vec_v,
+                   base + 2 * kL * DS);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    fetch(0, sm);
+    for (int t0 = 0, stage = 0; t0 < n; t0 += kL, stage ^= 1) {
         const int cnt = n - t0 < kL ? n - t0 : kL;
         const long long row = row0 + t0;
-        if (o) load_heads(in, in.q_off, row, cnt, h, D, Dp, DS, 1.0f, vec, sQ);
-        load_heads(in, in.k_off, row, cnt, h, D, Dp, DS, in.k_scale, vec, sK);
-        for (int i = threadIdx.x; i < kL * (cols >> 2); i += blockDim.x) {
-            const int tk = i / (cols >> 2), c = (i % (cols >> 2)) * 4;
-            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (tk < cnt && e0 + c < E) {
-                const float* p = in.src + (row + tk) * in.ld + in.v_off + (long long)h * E + e0 + c;
-                if (vec_v) {
-                    v = *reinterpret_cast<const float4*>(p);
-                } else {
-                    v.x = p[0];
-                    if (e0 + c + 1 < E) v.y = p[1];
-                    if (e0 + c + 2 < E) v.z = p[2];
-                    if (e0 + c + 3 < E) v.w = p[3];
-                }
-                if (in.silu) v.x = siluf_(v.x), v.y = siluf_(v.y), v.z = siluf_(v.z), v.w = siluf_(v.w);
-            }
-            *reinterpret_cast<float4*>(sV + tk * VS + c) = v;
+        float* sQ = sm + stage * stage_floats;
+        float* sK = sQ + kL * DS;
+        float* sV = sK + kL * DS;
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();  // this stage is here, and everybody is done with the other one
+        if (t0 + kL < n) fetch(t0 + kL, sm + (stage ^ 1) * stage_floats);
+        if (in.silu) {
+            if (o) silu_rows(sQ, Dp, DS);
+            silu_rows(sK, Dp, DS);
+            silu_rows(sV, cols, VS);
+            if (in.k_scale != 1.0f) turn_rows(in, row, cnt, D, DS, nullptr, sK);
+        } else {
+            turn_rows(in, row, cnt, D, DS, o ? sQ : nullptr, sK);
         }
         __syncthreads();
         float acc[2][2][4];
@@ -437,7 +477,6 @@ decay_chunk_kernel(DecayIn in, const float* __restrict__ pow_h, int pow_ld, cons
                 mma3(S[nt], a, bb);
             }
         }
-        __syncthreads();
     }
     if (fin < 0) return;
     float* sf = final_buf + ((long long)fin * H + h) * de;
@@ -527,13 +566,13 @@ extern "C" int llark_seq_decay_chunks(const float* src, long long ld, int q_off,
     const int cols = 16 * warps;
     auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
     const bool rows16 = ld % 4 == 0 && al(src);
-    const int vec = rows16 && D % 4 == 0 && q_off % 4 == 0 && k_off % 4 == 0 &&
-                    (n_rot == 0 || (n_rot % (interleaved ? 4 : 8) == 0 && al(cs)));
+    if (n_rot && !al(cs)) return LLARK_EINVAL;
+    const int vec = rows16 && D % 4 == 0 && q_off % 4 == 0 && k_off % 4 == 0;
     const int vec_v = rows16 && E % 4 == 0 && v_off % 4 == 0 && (!o || al(o));
     const dim3 grid((E + cols - 1) / cols, H, n_items);
 #define LLARK_DCHUNK(NT)                                                                                                 \
     do {                                                                                                                 \
-        const size_t smem = sizeof(float) * (size_t)(2 * kL * (8 * NT + 8) + kL * (cols + 8) + kL * kAS + kL + 4);       \
+        const size_t smem = sizeof(float) * (size_t)(2 * kL * (2 * (8 * NT + 8) + cols + 8) + kL * kAS + kL + 4);        \
         if (smem > 48 * 1024) {                                                                                          \
             cudaError_t e = cudaFuncSetAttribute(decay_chunk_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize,     \
                                                  (int)smem);                                                             \

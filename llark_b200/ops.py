@@ -808,14 +808,30 @@ def seq_glr_scan(src, q_off, f_off, v_off, lower, state, st, H, D, E):
 
 
 # linear attention with a fixed decay per head (csrc/seq_decay.cu)
-DECAY_CHUNK = 256         # rows per work item when a long prompt is scanned in chunks
+DECAY_CHUNKS = (128, 256, 384, 512, 768, 1024)  # rows per work item when a long prompt is scanned in chunks
 DECAY_CHUNK_MIN_LEN = 16  # shortest longest-request of a step that goes to the tensor-core kernel
 
 
+def decay_chunk_rows(lens, H, E):
+    """Rows per work item for prompts of `lens` tokens: None = one item per request, a single pass. Two blocks share one of the
+    148 SMs; a pass takes as long as its waves of blocks, the pass over local states less than half of the one with outputs."""
+    def waves(items):
+        blocks = items * H * ((E + 127) // 128)
+        return 0.6 if blocks <= 148 else -(-blocks // 296)
+
+    best, rows = waves(len(lens)) * max(lens), None
+    for L in DECAY_CHUNKS:
+        if L < max(lens):
+            t = waves(sum(-(-n // L) for n in lens)) * L * 1.45
+            if t <= (best if rows else 0.9 * best):  # of two equal ones the longer: fewer states between the passes
+                best, rows = t, L
+    return rows
+
+
 def decay_powers(decay, device):
-    """decay^0 .. decay^DECAY_CHUNK per head, fp32 [H, DECAY_CHUNK + 1] (powers taken in float64)."""
+    """decay^0, decay^1, ... up to the longest chunk per head, fp32 [H, n + 1] (powers taken in float64)."""
     d = torch.tensor([float(z) for z in decay], dtype=torch.float64)[:, None]
-    return torch.pow(d, torch.arange(DECAY_CHUNK + 1, dtype=torch.float64)[None, :]).to(device=device, dtype=torch.float32).contiguous()
+    return torch.pow(d, torch.arange(DECAY_CHUNKS[-1] + 1, dtype=torch.float64)[None, :]).to(device=device, dtype=torch.float32).contiguous()
 
 
 def seq_rotary_table(freq, st):
@@ -836,30 +852,36 @@ def seq_decay_scan(src, q_off, k_off, v_off, powers, state, st, H, D, E, freq=No
     """src fp32 [n_tok, ld] (q, k: H*D columns at q_off, k_off; v: H*E at v_off) -> o fp32 [n_tok, H*E] of S <- decay_h S + k v^T,
     o = S^T q; state fp32 [slots, H, D, E] read and written back; powers: decay_powers(). freq: rotary positions on q and k;
     k_scale: factor on k; silu: SiLU on q, k and v. Prompts go to the tensor-core kernel (three split TF32 products per
-    product, fp32 accuracy), in three passes over chunks of DECAY_CHUNK rows when there are too few (request, head) pairs to
+    product, fp32 accuracy), in three passes over chunks of rows when there are too few (request, head) pairs to
     fill the GPU; single tokens, short portions, wide heads and full_fp32 to the token-by-token kernel."""
     _req(src, torch.float32), _req(state, torch.float32), _req(powers, torch.float32)
     L = lib()
     o = torch.empty((st.n_tok, H * E), device=src.device, dtype=torch.float32)
     n_rot = 2 * freq.numel() if freq is not None else 0
-    head = (_p(src), src.stride(0), q_off, k_off, v_off, _p(seq_rotary_table(freq, st)) if n_rot else None, n_rot,
-            int(interleaved), float(k_scale), int(silu), _p(powers), powers.shape[1])
+    cs = _p(seq_rotary_table(freq, st)) if n_rot else None
+    inter, ks, silu, pw, pl = int(interleaved), float(k_scale), int(silu), _p(powers), powers.shape[1]
+    S = _p(state)
     if full_fp32 or st.max_len < DECAY_CHUNK_MIN_LEN or D > 128:
-        check(L.llark_seq_decay_rows(*head, _p(state), _p(state), _p(o), _p(st.cu), _p(st.lens_dev), _p(st.slot), _p(st.slot),
-                                     st.n_seq, st.max_len, H, D, E, _stream()), "seq_decay_rows")
+        check(L.llark_seq_decay_rows(_p(src), src.stride(0), q_off, k_off, v_off, cs, n_rot, inter, ks, silu, pw, pl, S, S, _p(o),
+                                     _p(st.cu), _p(st.lens_dev), _p(st.slot), _p(st.slot), st.n_seq, st.max_len, H, D, E,
+                                     _stream()), "seq_decay_rows")
         return o
-    if st.max_len <= DECAY_CHUNK or st.n_seq * H * ((E + 127) // 128) >= 4 * 148:
-        check(L.llark_seq_decay_chunks(*head, _p(state), _p(state), _p(o), _p(st.cu), _p(st.lens_dev), _p(st.slot), _p(st.slot),
-                                       st.n_seq, H, D, E, _stream()), "seq_decay_chunks")
+    rows = decay_chunk_rows(st.lens, H, E)
+    if rows is None:
+        check(L.llark_seq_decay_chunks(_p(src), src.stride(0), q_off, k_off, v_off, cs, n_rot, inter, ks, silu, pw, pl, S, S,
+                                       _p(o), _p(st.cu), _p(st.lens_dev), _p(st.slot), _p(st.slot), st.n_seq, H, D, E,
+                                       _stream()), "seq_decay_chunks")
         return o
-    ch = st.chunks(DECAY_CHUNK)
+    ch = st.chunks(rows)
     cstate = torch.empty((ch.n_items, H, D, E), device=src.device, dtype=torch.float32)
-    check(L.llark_seq_decay_chunks(*head, None, _p(cstate), None, _p(ch.row0), _p(ch.n), _p(ch.minus1), _p(ch.inner),
-                                   ch.n_items, H, D, E, _stream()), "seq_decay_chunks(local)")
-    check(L.llark_seq_decay_combine(_p(state), _p(cstate), _p(powers), powers.shape[1], _p(ch.n), _p(ch.seq_item0), _p(st.slot),
-                                    st.n_seq, H, D, E, _stream()), "seq_decay_combine")
-    check(L.llark_seq_decay_chunks(*head, _p(cstate), _p(state), _p(o), _p(ch.row0), _p(ch.n), _p(ch.index), _p(ch.last_slot),
-                                   ch.n_items, H, D, E, _stream()), "seq_decay_chunks(outputs)")
+    check(L.llark_seq_decay_chunks(_p(src), src.stride(0), q_off, k_off, v_off, cs, n_rot, inter, ks, silu, pw, pl, None,
+                                   _p(cstate), None, _p(ch.row0), _p(ch.n), _p(ch.minus1), _p(ch.inner), ch.n_items, H, D, E,
+                                   _stream()), "seq_decay_chunks(local)")
+    check(L.llark_seq_decay_combine(S, _p(cstate), pw, pl, _p(ch.n), _p(ch.seq_item0), _p(st.slot), st.n_seq, H, D, E,
+                                    _stream()), "seq_decay_combine")
+    check(L.llark_seq_decay_chunks(_p(src), src.stride(0), q_off, k_off, v_off, cs, n_rot, inter, ks, silu, pw, pl, _p(cstate), S,
+                                   _p(o), _p(ch.row0), _p(ch.n), _p(ch.index), _p(ch.last_slot), ch.n_items, H, D, E,
+                                   _stream()), "seq_decay_chunks(outputs)")
     return o
 
 

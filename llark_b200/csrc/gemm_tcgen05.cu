@@ -61,7 +61,8 @@ struct GemmParams {
     // fused epilogue (LlarkGemmEpilogue): 0 none, 1 quick-GELU, 2 RoPE on the first epi_i1 columns (head_dim 128,
     // position = row % epi_i0, epi_a / epi_b = cos / sin bf16 [S,128]), 3 SwiGLU backward (epi_a = gu bf16 [M, epi_ld]:
     // gate | up halves N apart; C receives dgate at column c and dup at column N + c), 5 squared ReLU, 6 gated ReLU (weight
-    // rows alternate gate, up: C column c = relu(acc column 2c) * acc column 2c + 1; C has N / 2 columns)
+    // rows alternate gate, up: C column c = relu(acc column 2c) * acc column 2c + 1; C has N / 2 columns), 7 the same with the
+    // clamped gated unit (epi_f0 = limit, epi_f1 = slope)
     int staged;      // 1 = staged (coalesced) epilogue, 0 = direct row-per-thread stores (see epilogue_dispatch)
     int group_m;     // m-blocks per rasterisation group (tile_coord): sized on the host so a group's A panel stays in L2
     int epi;

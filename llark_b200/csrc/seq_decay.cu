@@ -491,18 +491,42 @@ decay_chunk_kernel(DecayIn in, const float* __restrict__ pow_h, int pow_ld, cons
 
 // Between the two chunk passes: on entry chunk_state[w] is what chunk w builds from zero (not read for the last chunk of a
 // request), on exit the state it STARTS from: the request's stored state, then S <- decay^(rows of w) S + local_w.
+// Up to WB chunks' states are requested before the first is used; V adjacent entries per thread (16-byte accesses with V = 4).
+template <int V>
 __global__ void decay_combine_kernel(const float* __restrict__ state, float* __restrict__ chunk_state,
                                      const float* __restrict__ pow_h, int pow_ld, const int* __restrict__ item_n,
                                      const int* __restrict__ seq_item0, const int* __restrict__ slot, int H, long long de) {
+    constexpr int WB = 8;
     const int h = blockIdx.y, b = blockIdx.z;
     const int w0 = seq_item0[b], w1 = seq_item0[b + 1];
-    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < de; i += (long long)gridDim.x * blockDim.x) {
-        float S = state[((long long)slot[b] * H + h) * de + i];
-        for (int w = w0; w < w1; ++w) {
-            float* cs = chunk_state + ((long long)w * H + h) * de + i;
-            const float loc = w + 1 < w1 ? *cs : 0.f;
-            *cs = S;
-            S = fmaf(pow_h[(long long)h * pow_ld + item_n[w]], S, loc);
+    const long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * V;
+    if (i >= de) return;
+    auto ld = [](const float* p, float (&v)[V]) {
+        if constexpr (V == 4) {
+            const float4 x = *reinterpret_cast<const float4*>(p);
+            v[0] = x.x, v[1] = x.y, v[2] = x.z, v[3] = x.w;
+        } else {
+            v[0] = *p;
+        }
+    };
+    float S[V], loc[WB][V], p[WB];
+    ld(state + ((long long)slot[b] * H + h) * de + i, S);
+    for (int c0 = w0; c0 < w1; c0 += WB) {
+#pragma unroll
+        for (int u = 0; u < WB; ++u) {
+            p[u] = c0 + u < w1 ? pow_h[(long long)h * pow_ld + item_n[c0 + u]] : 0.f;
+            if (c0 + u + 1 < w1) ld(chunk_state + ((long long)(c0 + u) * H + h) * de + i, loc[u]);
+        }
+#pragma unroll
+        for (int u = 0; u < WB; ++u) {
+            if (c0 + u >= w1) break;
+            float* cs = chunk_state + ((long long)(c0 + u) * H + h) * de + i;
+            if constexpr (V == 4) *reinterpret_cast<float4*>(cs) = make_float4(S[0], S[1], S[2], S[3]);
+            else *cs = S[0];
+            if (c0 + u + 1 < w1) {
+#pragma unroll
+                for (int v = 0; v < V; ++v) S[v] = fmaf(p[u], S[v], loc[u][v]);
+            }
         }
     }
 }
@@ -599,7 +623,11 @@ extern "C" int llark_seq_decay_combine(const float* state, float* chunk_state, c
         !slot)
         return LLARK_EINVAL;
     const long long de = (long long)D * E;
-    const dim3 grid((unsigned)((de + 255) / 256), H, n_seq);
-    decay_combine_kernel<<<grid, 256, 0, st>>>(state, chunk_state, pow_h, pow_ld, item_n, seq_item0, slot, H, de);
+    const bool vec = de % 4 == 0 && ((reinterpret_cast<uintptr_t>(state) | reinterpret_cast<uintptr_t>(chunk_state)) & 15) == 0;
+    const dim3 grid((unsigned)((de / (vec ? 4 : 1) + 127) / 128), H, n_seq);
+    if (vec)
+        decay_combine_kernel<4><<<grid, 128, 0, st>>>(state, chunk_state, pow_h, pow_ld, item_n, seq_item0, slot, H, de);
+    else
+        decay_combine_kernel<1><<<grid, 128, 0, st>>>(state, chunk_state, pow_h, pow_ld, item_n, seq_item0, slot, H, de);
     return check_launch();
 }

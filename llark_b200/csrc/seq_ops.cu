@@ -18,11 +18,14 @@
 //   llark_seq_tanh_norm     y = tanh(alpha * x) * w + b -> ACT: an element-wise squashing that stands where others have a norm
 //   llark_seq_tanh_norm_add x_out = x + tanh(alpha * f) * w + b with f = a sublayer's result and / or the weighted sum of the
 //                           outputs of a token's chosen experts; optional ACT copy of the next sublayer's tanh norm of x_out
+//   llark_seq_layer_norm_add  x_out = x + layernorm(f) * w, f as in llark_seq_tanh_norm_add; optional ACT copy of the next
+//                           sublayer's layer norm of x_out or of x_out itself; also the plain layer norm of chosen rows
 //   llark_linear_rows       C = act(A W^T (+ bias)) for a handful of rows: weight-streaming, one or two output columns per warp
 //   llark_linear_simt       C = act(A W^T (+ bias)), any shape, tiled SIMT with fp32 accumulation (the fp32 mode's GEMM and the
 //                           fallback for shapes the TMA descriptors of the tcgen05 core cannot take)
 //                           act: LLARK_ACT_NONE, LLARK_ACT_RELU2 (squared ReLU), LLARK_ACT_RELU_GLU (weight rows alternate gate,
-//                           up: output column c = relu(column 2c) * column 2c + 1)
+//                           up: output column c = relu(column 2c) * column 2c + 1), LLARK_ACT_CLAMP_GLU (the same with the
+//                           clamped gated unit)
 #include <initializer_list>
 
 #include "common.cuh"

@@ -70,7 +70,7 @@ class BuvesunEngine(LayerListEngine):
         cfg = self.cfg
         cache = StateCache(self.device, n_slots=n_slots, positions=self.max_positions or 256)
         entries = []
-        for i, enters in cfg.layer_runs():
+        for i, _, enters in cfg.layer_runs():
             pk = self._packed[i]
             entries.append({"pk": pk, "enters": enters,
                             "mixer": MIXERS[MIXER_TYPES[cfg.layers[i].type]](pk["mixer"], cache, cfg.eps, self.act,

@@ -1,5 +1,5 @@
 """The step function shared by the layer-list decoders of the generation path (Kelutar, Golavik, Gubulorn, Tokatar,
-Manapel): one `step()` runs a PACKED batch (llark_b200.state_cache) -- requests that start, go on by a portion of their prompt or decode one token are
+Manapel, Buvesun): one `step()` runs a PACKED batch (llark_b200.state_cache) -- requests that start, go on by a portion of their prompt or decode one token are
 the same kernels with other numbers -- and returns fp32 logits for the rows that are asked for. A model's engine
 subclasses this and says how tokens become the residual stream (`_embed`), what its layers do to it (`_run_layers`) and
 how wanted rows become logits (`_logits`); slot handling, the step descriptor, validation and the order of things are

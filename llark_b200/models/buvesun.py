@@ -27,6 +27,7 @@ l<i>.mlp.e<j>.gate / up / down, l<i>.mlp.shared.gate / up / down.
 from dataclasses import dataclass, field
 from typing import List, Optional
 
+from llark_b200.models.layer_loop import layer_runs, read_loop
 from llark_b200.models.native import NativeCausalLM
 
 ARCHITECTURE = "Buvesun"
@@ -74,14 +75,10 @@ class BuvesunConfig:
             layers.append(BuvesunLayer(type=e["type"], mixer=mixer, mlp=dict(mlp) if mlp else None))
         if not layers:
             raise ValueError("a model needs at least one layer")
-        loop = d.get("loop")
-        if loop:
-            loop = {k: int(loop[k]) for k in ("start", "stop", "times")}
-            if not 0 <= loop["start"] < loop["stop"] <= len(layers) or loop["times"] < 1:
-                raise ValueError("loop: start .. stop - 1 must be layers, times at least 1")
         return cls(vocab=int(d["vocab"]), width=int(d["width"]), eps=float(d["norm"]["eps"]),
                    embedding_scale=float((d.get("embedding") or {}).get("scale", 1.0)),
-                   residual_mult=float(d.get("residual_mult", 1.0)), layers=layers, loop=loop or None,
+                   residual_mult=float(d.get("residual_mult", 1.0)), layers=layers,
+                   loop=read_loop(d.get("loop"), len(layers)),
                    eos_token_id=d.get("eos_token_id"), pad_token_id=d.get("pad_token_id"))
 
     def to_dict(self):
@@ -90,13 +87,8 @@ class BuvesunConfig:
                 "layers": [{"type": l.type, "mixer": l.mixer, "mlp": l.mlp} for l in self.layers]}
 
     def layer_runs(self):
-        """[(layer number, whether a pass of the loop begins with it)] in the order of execution."""
-        n = len(self.layers)
-        if not self.loop:
-            return [(i, False) for i in range(n)]
-        a, b = self.loop["start"], self.loop["stop"]
-        once = [(i, i == a) for i in range(a, b)]
-        return [(i, False) for i in range(a)] + once * self.loop["times"] + [(i, False) for i in range(b, n)]
+        """(layer, pass, first layer of a pass?) in the order the layers run; pass is None outside the loop."""
+        return layer_runs(self.loop, len(self.layers))
 
 
 class BuvesunForCausalLM(NativeCausalLM):

@@ -20,6 +20,7 @@ down.
 from dataclasses import dataclass, field
 from typing import List, Optional
 
+from llark_b200.models.layer_loop import layer_runs, read_loop
 from llark_b200.models.native import NativeCausalLM
 
 ARCHITECTURE = "Golavik"
@@ -62,27 +63,14 @@ class GolavikConfig:
         width, groups = int(d["width"]), int(d["norm"].get("groups", 1))
         if groups < 1 or width % groups:
             raise ValueError("norm.groups must divide width")
-        loop = d.get("loop")
-        if loop is not None:
-            loop = {k: int(loop[k]) for k in ("start", "stop", "times")}
-            if not (0 <= loop["start"] <= loop["stop"] <= len(layers)) or loop["times"] < 1:
-                raise ValueError("loop must name a range of layers and a positive number of passes")
-            if loop["start"] == loop["stop"]:
-                loop = None
+        loop = read_loop(d.get("loop"), len(layers))
         return cls(vocab=int(d["vocab"]), width=width, eps=float(d["norm"]["eps"]), groups=groups,
                    taps=int(d["canon"]["taps"]), layers=layers, loop=loop, eos_token_id=d.get("eos_token_id"),
                    pad_token_id=d.get("pad_token_id"))
 
     def layer_runs(self):
         """(layer, pass, first layer of a pass?) in the order the layers run; pass is None outside the loop."""
-        n = len(self.layers)
-        if self.loop is None:
-            return [(i, None, False) for i in range(n)]
-        a, b, times = self.loop["start"], self.loop["stop"], self.loop["times"]
-        runs = [(i, None, False) for i in range(a)]
-        for t in range(times):
-            runs += [(i, t, i == a) for i in range(a, b)]
-        return runs + [(i, None, False) for i in range(b, n)]
+        return layer_runs(self.loop, len(self.layers))
 
     def to_dict(self):
         return {"architecture": ARCHITECTURE, "vocab": self.vocab, "width": self.width,

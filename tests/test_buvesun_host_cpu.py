@@ -31,12 +31,13 @@ def test_config_round_trip_and_layer_runs():
     assert (c.vocab, c.width, c.eps, c.embedding_scale, c.residual_mult) == (11, 12, 1e-5, 2.0, 0.4)
     assert c.layers[1].mlp is None and c.loop == {"start": 1, "stop": 3, "times": 2}
     assert BuvesunConfig.from_dict(json.loads(json.dumps(c.to_dict()))).to_dict() == c.to_dict()
-    assert c.layer_runs() == [(0, False), (1, True), (2, False), (1, True), (2, False)] == bo.layer_runs(_cfg())
+    assert [(i, f) for i, _, f in c.layer_runs()] == [(0, False), (1, True), (2, False), (1, True), (2, False)] == bo.layer_runs(_cfg())
+    assert [t for _, t, _ in c.layer_runs()] == [None, 0, 0, 1, 1]
     for loop, runs in ((None, [(0, False), (1, False), (2, False)]),
                        ({"start": 0, "stop": 1, "times": 3}, [(0, True), (0, True), (0, True), (1, False), (2, False)]),
                        ({"start": 2, "stop": 3, "times": 1}, [(0, False), (1, False), (2, True)])):
         d = dict(_cfg(), loop=loop)
-        assert BuvesunConfig.from_dict(d).layer_runs() == runs == bo.layer_runs(d)
+        assert [(i, f) for i, _, f in BuvesunConfig.from_dict(d).layer_runs()] == runs == bo.layer_runs(d)
 
 
 @pytest.mark.parametrize("bad", [
@@ -47,7 +48,7 @@ def test_config_round_trip_and_layer_runs():
     lambda d: d["layers"][0]["mixer"].update(decay=[0.5]),              # one per head
     lambda d: d["layers"][1]["mixer"]["right"].update(decay=[0.5, 1.5, 0.1]),
     lambda d: d["loop"].update(stop=4),
-    lambda d: d["loop"].update(start=3),
+    lambda d: d["loop"].update(start=-1),
     lambda d: d["loop"].update(times=0),
 ])
 def test_config_validation(bad):
